@@ -99,7 +99,9 @@ int exl3_embed_hashed(const int* ids, const int* tok_pos, const int* tok_seq, co
 // The step between an attention's joint input projection and the attention itself (see qk_prep.cu).
 //   x [T, ld] holds per token nh query heads (at q_off), nkv key heads (k_off) of hd features and nkv value heads
 //   (v_off, or < 0 for none) of hdv features.  norm: 0 none, 1 divide a query/key head by its root mean square,
-//   2 the same times q_w / k_w [hd].  rot > 0: rotary encoding of the first rot features (layout 0: feature i with
+//   2 the same times q_w / k_w [hd], 3 all query heads (all key heads) of a token together divided by their root mean
+//   square, times q_w [nh * hd] / k_w [nkv * hd].  temp_every > 0: queries at position p are multiplied by
+//   1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).  nkv 0: queries only (v_off < 0, no cache).  rot > 0: rotary encoding of the first rot features (layout 0: feature i with
 //   i + rot / 2; 1: feature 2i with 2i + 1), sines and cosines times mscale.  Keys are then multiplied by k_mul.
 //   mix_lambda != null: v <- (1 - lambda) v + lambda v_src[t] (v_src [T, v_src_ld], its own type).
 //   Queries go to q_out [T, nh * hd_pad]; keys and values to the paged cache (k_pool / v_pool, rows of hd_pad /
@@ -110,7 +112,7 @@ int exl3_qk_prep(const void* x, int x_dtype, int64_t ld, int q_off, int k_off, i
                  float k_mul, const void* mix_lambda, int lambda_dtype, const void* v_src, int v_src_dtype,
                  int64_t v_src_ld, const int* tok_pos, const int* tok_seq, const int* block_table, int bt_stride,
                  int page, void* q_out, int q_out_dtype, void* k_out, int k_out_dtype, void* k_pool, void* v_pool,
-                 int pool_dtype, cudaStream_t stream);
+                 int pool_dtype, float temp_coef, float temp_every, cudaStream_t stream);
 
 // Token shift: for s < n_mix, out[s][t] = h[t] + (h[t - 1] - h[t]) * mu[s]; the row before a row's first token of
 // this step comes from prev[slot] (float32 [slots, H], zero for a new sequence), which is then set to the row's last
@@ -267,7 +269,7 @@ int exl3_gemm_pair_ss_blocks(int N);
 // 4) and merge them in shared memory; 2: a cluster of two blocks (at most 8 chunks, the first block merging, the
 // second one's records read out of its shared memory); no scratch in either.  twins 2 (with in_block 1 or 2, an even
 // head_split and groups of up to 8 heads): two groups of query heads of a kv head per block, walking the same pages
-// out of the same rings, 8 computing warps.  See attention_decode.cu.
+// out of the same rings, 8 computing warps.  sink_vals and dist as in exl3_attn_tokens_opt.  See attention_decode.cu.
 int exl3_attn_decode_supported(int dtype, int T, int nh, int nkv, int hd, int page, int split_keys, int max_splits);
 int exl3_attn_decode_status();
 int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, void* k_pool, void* v_pool,
@@ -275,7 +277,7 @@ int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, void* k_poo
                      const int* tok_seq, int T, int nh, int nkv, int hd, int page, int window, int chunk, int sink,
                      float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes, const float* inv_freq,
                      const float* inv_freq_lo, int rot, float pos_scale, int write_new, int head_split, int in_block,
-                     int twins, cudaStream_t stream);
+                     int twins, const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream);
 
 int exl3_argmax(const float* logits, int* out, int R, int V, void* scratch, size_t scratch_bytes,
                 cudaStream_t stream);
@@ -301,7 +303,8 @@ int exl3_tanh_norm_add(float* h, const void* a, int a_dtype, const void* b, int 
 // A routed feed-forward (see moe.cu).  exl3_moe_route: wr float32 [E + extra, W]; idx int32 and wt float32 [T, top];
 // gate_out float32 [T] = sigmoid of the extra row.  exl3_moe_plan: order int32 [P], plan int32 [4 + 3 * max tiles].
 // exl3_moe_gemm: out[p] = act(W[e(p)] A[p / a_div]) for the planned pairs, W [n_experts, N, K]; act 0 none, 1 gelu
-// (exact), 2 gelu by the tanh formula, 3 silu.  exl3_moe_combine: the weighted sum, float32 [T, H]; picks from
+// (exact), 2 gelu by the tanh formula, 3 silu, 4 the square of relu.  score_kind: 0 softmax, 1 sigmoid, + 2 groups scored
+// by their two largest, 4 the softmax over the picks alone (corr is then a bias of the logits).  exl3_moe_combine: the weighted sum, float32 [T, H]; picks from
 // n_experts on stand for the input x itself; shared (any type) is added times gate (null: as it is).
 // exl3_moe_gemv: the same product for plans of tiles of at most exl3_moe_gemv_rows() rows (decode), bfloat16 A and W.
 // exl3_moe_gather + exl3_moe_gemm_tc (moe_tc.cu): rows of x in the plan's order, and the product on tcgen05 tensor
@@ -329,6 +332,11 @@ int exl3_moe_gemm(const void* A, int a_dtype, int64_t lda, int a_div, const void
 int exl3_moe_combine(const float* y, const int* idx, const float* wt, const void* x, int x_dtype, int64_t ldx,
                      const void* shared, int shared_dtype, const float* gate, float* out, int T, int H, int top,
                      int n_experts, cudaStream_t stream);
+// The weighted sum followed by an RMS norm of it that is added to the residual: h += v / rms(v) * w (w float32) and, with
+// x given, x = h in bfloat16.
+int exl3_moe_combine_norm(const float* y, const int* idx, const float* wt, const void* shared, int shared_dtype,
+                          const float* gate, float* h, const float* w, float eps, void* x, int T, int H, int top,
+                          int n_experts, cudaStream_t stream);
 
 // Heads of several maps (see diff_attn.cu): rotation, widened queries and the cache write; and the combination of
 // two maps' outputs.
@@ -340,14 +348,17 @@ int exl3_diff_combine(const void* a, int a_dtype, int a_row, const void* gate, i
                       float lambda, float eps, float mult, void* out, int out_dtype, int out_row, int T, int heads,
                       int dv, cudaStream_t stream);
 
-// exl3_attn_tokens_wide with three more options: with a window, keys at positions below keep_first stay visible; softcap > 0
+// exl3_attn_tokens_wide with four more options: with a window, keys at positions below keep_first stay visible; softcap > 0
 // replaces a score s (after the scale) by softcap * tanh(s / softcap); sink_vals [heads] (float32, with sink) are the
-// sink's scores per query head instead of 0.  max_splits must count the chunks of the kept keys too.
+// sink's scores per query head instead of 0; dist (dist_len > 0): biases per query head and distance, added to the scores
+// (after scale and cap) of keys less than dist_len positions back, a row per head of dist_len + 2 * DIST_PAD floats
+// (common.cuh).  max_splits must count the chunks of the kept keys too.
 int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* out, int out_f32, int dtype, const void* k_pool,
                          const void* v_pool, const int* block_table, int bt_stride, const int* tok_pos,
                          const int* tok_seq, int T, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                          int window, int chunk, int sink, float scale, int split_keys, int max_splits, float* scratch,
-                         size_t scratch_bytes, int keep_first, float softcap, const float* sink_vals, cudaStream_t stream);
+                         size_t scratch_bytes, int keep_first, float softcap, const float* sink_vals, const float* dist,
+                         int dist_len, cudaStream_t stream);
 
 // rows of gu are [gate (I) | up (I)], ld elements apart: out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit)
 // and u = clamp(up, -limit, limit).
@@ -391,7 +402,14 @@ int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int T, void* o
                              int64_t n_pool_rows, const int* block_table, int bt_stride, const int* row_start,
                              const int* row_pos0, const int* tile_seq, const int* tile_q0, int n_tiles, int nh, int nkv,
                              int hd, int page, int window, int chunk, int sink, float scale, int variant, int keep_first,
-                             float softcap, const float* sink_vals, cudaStream_t stream);
+                             float softcap, const float* sink_vals, const float* dist, int dist_len,
+                             cudaStream_t stream);
+// h[t] = table[ids[t]] * scale + a sinusoid of position tok_pos[t] (entry 2i: sin(p f_i), 2i + 1: cos(p f_i), f given as
+// float32 and what float32 lost, ceil(H / 2) each), then, with norm_w (float32 [H]) given, h / sqrt(mean(h^2) + eps) *
+// norm_w; float32, and in bfloat16 into x when x is given (see sinusoid_embed.cu).
+int exl3_embed_sinusoid(const int* ids, const int* tok_pos, const void* table, int dtype, float scale, const float* f_hi,
+                        const float* f_lo, const float* norm_w, float eps, float* h, void* x, int T, int H, int V,
+                        cudaStream_t stream);
 // y[M, N] (float32) = x[M, K] . w[N, K]^T (+ bias) for a handful of output features and many rows; x, w and bias of one
 // type, K and the pitch of x multiples of 16 bytes.
 int exl3_gemm_few_out(const void* x, int64_t ldx, const void* w, const void* bias, float* y, int in_dtype, int M, int N,

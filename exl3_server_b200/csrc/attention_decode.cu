@@ -49,6 +49,9 @@
 // the projection has finished (programmatic dependent launch).  This is for
 // steps in which every sequence brings one token.
 //
+// Options: a sink in the softmax's denominator (of score 0, or of a score per query head: sink_vals), and biases per
+// query head and distance added to the scaled scores of keys less than dist_len positions back (common.cuh, DIST_PAD).
+//
 // Cache layout: pool[page][kv_head][slot][head_dim], page = block_table[row][pos / page_size].
 #include "api.h"
 #include "common.cuh"
@@ -182,6 +185,13 @@ __device__ inline uint32_t ad_pack(float lo, float hi) {
 // heads of the same kv head: warp w and warp AD_WARPS + w walk the same chunk out of the same ring of pages, each
 // with its own group's queries, so that a page comes into shared memory once for both and a scheduler has two
 // warps to issue from.  A stage is free when both have read it (the barrier counts TW arrivals).
+struct AdOpts {
+  const float* sink_vals;                                // per query head, natural units; null: 0
+  const float* dist;                                     // biases per query head and distance; dist_len 0: none
+  int dist_len;
+  float dist_mul;                                        // 1 / scale: the biases join the scores before the scale
+};
+
 template <int HD, int NC, int TW>
 __global__ void __launch_bounds__((TW + 1) * AD_WARPS * 32, 1)
 attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
@@ -192,7 +202,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
                    int split_keys, int max_splits, float* __restrict__ scratch, int* __restrict__ counters,
                    const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, float pos_scale,
                    int rotate, int write_new,
-                   __nv_bfloat16* __restrict__ k_pool, __nv_bfloat16* __restrict__ v_pool, int kv_rep, int in_block) {
+                   __nv_bfloat16* __restrict__ k_pool, __nv_bfloat16* __restrict__ v_pool, int kv_rep, int in_block,
+                   AdOpts opts) {
   // nkv counts groups of query heads that are worked on together.  With kv_rep = 2 the query heads of a kv head
   // are two such groups (g and g + 1 read kv head g / 2): twice the work items and two merges of half the size,
   // for steps with few tokens, where a single warp's merge of a wide group is what takes the time.
@@ -272,6 +283,10 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
 
   const int G = nh / nkv;
   const int rec = HD + 2;
+  // the sink's term of a head's sum, with m the maximum the sum is kept against
+  auto sink_term = [&](int head, float m) {
+    return ad_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m);
+  };
   auto chunks_of = [&](int t) { return s_cum[t + 1] - s_cum[t]; };
   auto base_of = [&](int t, int g) { return nkv * s_cum[t] + g * chunks_of(t); };   // index of chunk 0 of (t, g)
   // This warp's share: chunks i0 .. i1 - 1 of the list ordered by token, kv head, chunk: an equal contiguous share
@@ -521,7 +536,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
           ll += lv[n * n_rec + s2] * w;
         }
         ll = warp_sum(ll);
-        if (sink) ll += ad_exp2(-M);
+        if (sink) ll += sink_term(mg * G + n0 + n, M);
         if (nn == n) my_ll = ll;
       }
     }
@@ -655,6 +670,22 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         }
       }
       const int key0 = pi * KS;
+      if (opts.dist_len > 0 && s_pos[t] - (key0 + KS - 1) < opts.dist_len) {
+        // the biases of the keys that are near enough
+        const int back0 = s_pos[t] - key0 - gl;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            const float* tab = dist_row(opts.dist, opts.dist_len, g * G + min(8 * c + 2 * tl + h, G - 1)) + back0;
+#pragma unroll
+            for (int a = 0; a < MT; ++a) {
+              s[c][a][h] = fmaf(__ldg(tab - 16 * a), opts.dist_mul, s[c][a][h]);
+              s[c][a][h + 2] = fmaf(__ldg(tab - 16 * a - 8), opts.dist_mul, s[c][a][h + 2]);
+            }
+          }
+        }
+      }
       if (key0 < c_lo || key0 + KS > c_hi) {
 #pragma unroll
         for (int a = 0; a < MT; ++a) {
@@ -760,7 +791,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         dot += __shfl_xor_sync(0xffffffffu, dot, 2);
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          const float sc = __shfl_sync(0xffffffffu, dot, (2 * tl + h) * 4) * scale_log2;
+          float sc = __shfl_sync(0xffffffffu, dot, (2 * tl + h) * 4) * scale_log2;
+          if (opts.dist_len > 0)
+            sc += __ldg(dist_row(opts.dist, opts.dist_len, g * G + min(8 * c + 2 * tl + h, G - 1))) * 1.4426950408889634f;
           const float mn = fmaxf(m[c][h], sc);
           const float corr = ad_exp2(m[c][h] - mn);              // 0 when the cache held no key of this chunk
           const uint32_t pp = ad_pack(ad_exp2(sc - mn), 0.0f);   // rounded as the other probabilities are
@@ -795,8 +828,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         const int head = g * G + n;
         if (n_rec == 1) {
           __nv_bfloat16* dst = out + ((int64_t)t * nh + head) * HD;
-          // a sink is one more key of score 0 without a value: a term exp2(0 - m) in the sum
-          const float inv = 1.0f / (sink ? l[c][h] + ad_exp2(-m[c][h]) : l[c][h]);
+          // a sink is one more key without a value: a term in the sum
+          const float inv = 1.0f / (sink ? l[c][h] + sink_term(head, m[c][h]) : l[c][h]);
 #pragma unroll
           for (int d = 0; d < NJ; ++d) {
             dst[16 * d + gl] = __float2bfloat16(o[c][d][h] * inv);
@@ -860,7 +893,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
           w[s2] = s2 < n_rec ? ad_exp2(rec_at(hb, s2, HD) - M) : 0.0f;
           ll += s2 < n_rec ? rec_at(hb, s2, HD + 1) * w[s2] : 0.0f;
         }
-        if (sink) ll += ad_exp2(-M);
+        if (sink) ll += sink_term(g_blk * G + n, M);
         __nv_bfloat16* dst = out + ((int64_t)t_blk * nh + g_blk * G + n) * HD;
 #pragma unroll
         for (int e = 0; e < HD / 32; ++e) {
@@ -969,8 +1002,13 @@ extern "C" int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, 
                                 int sink,
                                 float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes,
                                 const float* inv_freq, const float* inv_freq_lo, int rot, float pos_scale,
-                                int write_new, int head_split, int in_block, int twins, cudaStream_t stream) {
+                                int write_new, int head_split, int in_block, int twins, const float* sink_vals,
+                                const float* dist, int dist_len, cudaStream_t stream) {
   if (T == 0) return 0;
+  if (dist_len < 0 || (dist_len > 0 && dist == nullptr) || (sink_vals != nullptr && !sink)) {
+    set_error("attn_decode: a table of %d distance biases is missing, or sink scores come without the sink", dist_len);
+    return ERR_BAD_ARGUMENT;
+  }
   if (in_block < 0 || in_block > 2 || (in_block && (max_splits < 1 || max_splits > in_block * AD_WARPS))) {
     set_error("attn_decode: in_block is 0, 1 (a block merges up to %d chunks of a (token, group of heads) itself) or 2 "
               "(a cluster of two blocks, up to %d); got %d with %d chunks", AD_WARPS, 2 * AD_WARPS, in_block, max_splits);
@@ -1026,6 +1064,11 @@ extern "C" int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, 
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     if (sms < 1) sms = 1;
   }
+  AdOpts opts;
+  opts.sink_vals = sink_vals;
+  opts.dist = dist;
+  opts.dist_len = dist_len;
+  opts.dist_mul = 1.0f / scale;
   // a stage is a page (heads of 64) or half a page (heads of 128): the copy's box has as many rows
   const int box_rows = hd == 64 ? 64 : 32;
   CUtensorMap map_k, map_v;
@@ -1051,7 +1094,7 @@ extern "C" int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, 
              static_cast<const __nv_bfloat16*>(q), q_row_stride, static_cast<__nv_bfloat16*>(out), block_table,  \
              bt_stride, tok_pos, tok_seq, T, nh, groups, window, chunk, sink, scale * 1.4426950408889634f, split_keys,        \
              max_splits, records, counters, inv_freq, inv_freq_lo, pos_scale, rot != 0 ? 1 : 0, write_new ? 1 : 0,            \
-             static_cast<__nv_bfloat16*>(k_pool), static_cast<__nv_bfloat16*>(v_pool), head_split, in_block)
+             static_cast<__nv_bfloat16*>(k_pool), static_cast<__nv_bfloat16*>(v_pool), head_split, in_block, opts)
   const bool wide = nh / groups > 8;                       // more than one block of 8 query heads per group
   if (hd == 64) { if (wide) EXL3_AD_LAUNCH(64, 2, 1); else if (twins == 2) EXL3_AD_LAUNCH(64, 1, 2); else EXL3_AD_LAUNCH(64, 1, 1); }
   else { if (wide) EXL3_AD_LAUNCH(128, 2, 1); else if (twins == 2) EXL3_AD_LAUNCH(128, 1, 2); else EXL3_AD_LAUNCH(128, 1, 1); }

@@ -175,12 +175,21 @@ __device__ inline uint32_t fa_pack(float lo, float hi) {
 // What a block needs to know of a tile of 128 queries.
 // Options beyond the plain causal softmax.  keep_first: with a window, the keys at positions below it stay visible.
 // cap_in > 0: a raw score s becomes tanh(s * cap_in) and is multiplied by cap_log2 (= cap * log2 e) instead of the
-// scale.  sink_vals: the sink's score per query head (natural units), or null for 0.
+// scale.  sink_vals: the sink's score per query head (natural units), or null for 0.  dist_len > 0: biases per head and
+// distance for keys less than dist_len positions back (see DIST_PAD); dist_mul brings them to the units in which the
+// scores stand before the scale (1 / scale) or after the tanh (1 / cap).
 struct FaOpts {
   int keep_first;
   float cap_in, cap_log2;
   const float* sink_vals;
+  const float* dist;
+  int dist_len;
+  float dist_mul;
 };
+// Whether a page of keys from key0 on holds a key with a bias for one of a warp's 32 queries from position p0 on.
+__device__ inline bool fa_near(int key0, int p0, int dist_len) {
+  return p0 - (key0 + FA_BK - 1) < dist_len && p0 + 31 >= key0;
+}
 // Pages from the sequence's start that a tile walks before the pages of its window: those that hold kept first keys
 // and lie before the window's first page.
 __device__ inline int fa_kept_pages(int window, int keep_first, int page_lo) {
@@ -444,6 +453,15 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
           for (int c = 0; c < 32; ++c) sr[h][c] = __float_as_uint(fa_tanh(__uint_as_float(sr[h][c]) * opts.cap_in));
       }
+      if (opts.dist_len > 0 && fa_near(key0, p_first + warp * 32, opts.dist_len)) {
+        // the biases of this row's distances p - key: neighbouring lanes read neighbouring entries
+        const float* tab = dist_row(opts.dist, opts.dist_len, head) + (p - key0);
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            sr[h][c] = __float_as_uint(fmaf(__ldg(tab - (h * 32 + c)), opts.dist_mul, __uint_as_float(sr[h][c])));
+      }
       if (need_mask) {
         int lo_key = (window > 0) ? p - window : -1;          // keys <= lo_key are out of the window
         if (chunk > 0) lo_key = max(lo_key, p / chunk * chunk - 1);   // or before the query's block of positions
@@ -701,6 +719,14 @@ attn_prefill_tc4_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
           for (int c = 0; c < 32; ++c) sr[h][c] = __float_as_uint(fa_tanh(__uint_as_float(sr[h][c]) * opts.cap_in));
       }
+      if (opts.dist_len > 0 && fa_near(key0, p_first + warp * 32, opts.dist_len)) {
+        const float* tab = dist_row(opts.dist, opts.dist_len, head) + (p - key0);
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            sr[h][c] = __float_as_uint(fmaf(__ldg(tab - (h * 32 + c)), opts.dist_mul, __uint_as_float(sr[h][c])));
+      }
       if (need_mask) {
         int lo_key = (window > 0) ? p - window : -1;
         if (chunk > 0) lo_key = max(lo_key, p / chunk * chunk - 1);
@@ -846,14 +872,19 @@ extern "C" int exl3_attn_prefill_tc_status() {
 // q: rows of the fused q|k|v buffer (row stride q_row_stride elements, T rows in all); tiles of 128 queries.
 // n_pool_rows = pages * kv_heads * 64 rows of head_dim in each of k_pool and v_pool.
 // The options of the general form: with a window, keys at positions below keep_first stay visible; softcap > 0 replaces a
-// scaled score s by softcap * tanh(s / softcap); sink_vals [heads] (float32, with sink) are the sink's scores.
+// scaled score s by softcap * tanh(s / softcap); sink_vals [heads] (float32, with sink) are the sink's scores; dist: a
+// bias per head and distance added to the scores (after the cap) of keys less than dist_len positions back.
 extern "C" int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int T, void* out, const void* k_pool,
                                         const void* v_pool, int64_t n_pool_rows, const int* block_table, int bt_stride,
                                         const int* row_start, const int* row_pos0, const int* tile_seq,
                                         const int* tile_q0, int n_tiles, int nh, int nkv, int hd, int page, int window,
                                         int chunk, int sink, float scale, int variant, int keep_first, float softcap,
-                                        const float* sink_vals, cudaStream_t stream) {
+                                        const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
+  if (dist_len < 0 || (dist_len > 0 && dist == nullptr)) {
+    set_error("attn_prefill_tc: a table of %d distance biases is missing", dist_len);
+    return ERR_BAD_ARGUMENT;
+  }
   if (keep_first < 0 || softcap < 0.0f || !(scale > 0.0f) || (sink_vals != nullptr && !sink)) {
     set_error("attn_prefill_tc: keep_first %d, softcap %g, scale %g: none may be negative, and sink scores need the sink",
               keep_first, (double)softcap, (double)scale);
@@ -864,6 +895,9 @@ extern "C" int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int
   opts.cap_in = softcap > 0.0f ? scale / softcap : 0.0f;
   opts.cap_log2 = softcap * 1.4426950408889634f;
   opts.sink_vals = sink_vals;
+  opts.dist = dist;
+  opts.dist_len = dist_len;
+  opts.dist_mul = softcap > 0.0f ? 1.0f / softcap : 1.0f / scale;
   if (!exl3_attn_prefill_tc_supported(DT_BF16, hd, page)) {
     set_error("attn_prefill_tc: needs bfloat16, head_dim 64 or 128 and pages of 64, got head_dim %d page %d", hd, page);
     return ERR_UNSUPPORTED;
@@ -930,5 +964,5 @@ extern "C" int exl3_attn_prefill_tc(const void* q, int64_t q_row_stride, int T, 
                                     int chunk, int sink, float scale, int variant, cudaStream_t stream) {
   return exl3_attn_prefill_tc_opt(q, q_row_stride, T, out, k_pool, v_pool, n_pool_rows, block_table, bt_stride, row_start,
                                   row_pos0, tile_seq, tile_q0, n_tiles, nh, nkv, hd, page, window, chunk, sink, scale,
-                                  variant, 0, 0.0f, nullptr, stream);
+                                  variant, 0, 0.0f, nullptr, nullptr, 0, stream);
 }

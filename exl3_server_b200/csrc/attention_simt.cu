@@ -30,12 +30,14 @@
 //              counted from the start of the sequence), on top of the causal bound and the window;
 //   sink:      one is added to the softmax's denominator, as if there were one more key with score 0 and a value
 //              of zero: p_j = exp(s_j) / (1 + sum_j exp(s_j)).
-// The entry point with every option (exl3_attn_tokens_opt) takes three more:
+// The entry point with every option (exl3_attn_tokens_opt) takes four more:
 //   keep_first > 0: with a window, the keys at positions below keep_first stay visible to every later query (at their
 //              true positions): j is seen when j <= pos and (pos - j < window or j < keep_first);
 //   softcap > 0: s <- softcap * tanh(s / softcap) after the scale;
 //   sink_vals: with sink, the sink's score per query head (not scaled, not capped) instead of 0:
-//              p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j)).
+//              p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j));
+//   dist:      s <- s + dist_h[pos - j] after the scale and the cap, for keys up to dist_len - 1 positions back (a
+//              table per query head; nothing is added further back).  Its layout is common.cuh's DIST_PAD.
 #include "api.h"
 #include "common.cuh"
 
@@ -108,7 +110,7 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
                    const int* __restrict__ tok_seq, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                    int window, int chunk, int sink, float scale, int split_keys, int max_splits,
                    float* __restrict__ scratch, int* __restrict__ counters, int lpk, int out_f32, int keep_first,
-                   float softcap, const float* __restrict__ sink_vals) {
+                   float softcap, const float* __restrict__ sink_vals, const float* __restrict__ dist, int dist_len) {
   constexpr int VEC = Elem<T>::vec;
   constexpr int NA = R * VEC;
   constexpr int U = R == 1 ? 4 : (R == 2 ? 2 : 1);  // key groups whose loads are issued together
@@ -220,6 +222,11 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
               for (int o = lpk >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
               if (valid[u]) {
                 s = cap_mul > 0.0f ? cap_mul * tanhf(s * cap_in) : s * scale_eff;
+                if (dist_len > 0) {
+                  const int back = pos - (pi * page + jj0 + u * kpw);
+                  if (back < dist_len && h0 + hh < G)
+                    s = fmaf(__ldg(dist_row(dist, dist_len, g * G + h0 + hh) + back), SoftmaxExp<T>::prescale, s);
+                }
                 const float mn = fmaxf(m[hh], s);
                 const float corr = SoftmaxExp<T>::exp(m[hh] - mn);    // exp(-inf) = 0 on the first key
                 const float p = SoftmaxExp<T>::exp(s - mn);
@@ -375,7 +382,8 @@ static int launch_tokens(const void* q, int64_t q_row_stride, void* out, const v
                          const void* v_pool, const int* block_table, int bt_stride, const int* tok_pos,
                          const int* tok_seq, int T_, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                          int window, int chunk, int sink, float scale, int split_keys, int max_splits, float* scratch, int lpk,
-                         int out_f32, int keep_first, float softcap, const float* sink_vals, cudaStream_t stream) {
+                         int out_f32, int keep_first, float softcap, const float* sink_vals, const float* dist, int dist_len,
+                         cudaStream_t stream) {
   const size_t smem = ((size_t)ATT_WARPS * GT * (hdv + 2) + 2 * (size_t)max_splits) * sizeof(float);
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(attn_tokens_kernel<T, GT, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -395,7 +403,7 @@ static int launch_tokens(const void* q, int64_t q_row_stride, void* out, const v
              static_cast<const T*>(q), q_row_stride, static_cast<T*>(out), static_cast<const T*>(k_pool),
              static_cast<const T*>(v_pool), block_table, bt_stride, tok_pos, tok_seq, nh, nkv, hd, hdv, kv_row, v_row, page,
              window, chunk, sink, scale, split_keys, max_splits, scratch, counters, lpk, out_f32, keep_first, softcap,
-             sink_vals);
+             sink_vals, dist, dist_len);
   int rc = launch_status("attn_tokens");
   if (rc) return rc;
   if (max_splits > 1 && !fused_merge) {
@@ -411,7 +419,7 @@ static int dispatch(const void* q, int64_t q_row_stride, void* out, const void* 
                     const int* block_table, int bt_stride, const int* tok_pos, const int* tok_seq, int T_,
                     int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page, int window, int chunk, int sink,
                     float scale, int split_keys, int max_splits, float* scratch, int out_f32, int keep_first, float softcap,
-                    const float* sink_vals, cudaStream_t stream) {
+                    const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream) {
   constexpr int VEC = Elem<T>::vec;
   const int vecs = ceil_div(max(hd, hdv), VEC);       // 16-byte pieces of the wider of a key row and a value row
   int lpk = 1;
@@ -421,7 +429,8 @@ static int dispatch(const void* q, int64_t q_row_stride, void* out, const void* 
 #define EXL3_ATT(GT, RR)                                                                                 \
   return launch_tokens<T, GT, RR>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos, \
                                   tok_seq, T_, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, \
-                                  split_keys, max_splits, scratch, lpk, out_f32, keep_first, softcap, sink_vals, stream)
+                                  split_keys, max_splits, scratch, lpk, out_f32, keep_first, softcap, sink_vals, \
+                                  dist, dist_len, stream)
   if (R == 1) {
     if (G == 1) EXL3_ATT(1, 1);
     if (G == 2) EXL3_ATT(2, 1);
@@ -461,8 +470,13 @@ extern "C" int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* o
                                     int bt_stride, const int* tok_pos, const int* tok_seq, int T, int nh, int nkv,
                                     int hd, int hdv, int kv_row, int v_row, int page, int window, int chunk, int sink,
                                     float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes,
-                                    int keep_first, float softcap, const float* sink_vals, cudaStream_t stream) {
+                                    int keep_first, float softcap, const float* sink_vals, const float* dist, int dist_len,
+                                    cudaStream_t stream) {
   if (T == 0) return 0;
+  if (dist_len < 0 || (dist_len > 0 && dist == nullptr)) {
+    set_error("attn_tokens: a table of %d distance biases is missing", dist_len);
+    return ERR_BAD_ARGUMENT;
+  }
   if (keep_first < 0 || softcap < 0.0f || (sink_vals != nullptr && !sink)) {
     set_error("attn_tokens: keep_first %d and softcap %g must not be negative, and sink scores need the sink", keep_first,
               (double)softcap);
@@ -494,11 +508,12 @@ extern "C" int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* o
   if (dtype == DT_F32)
     return dispatch<float>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos, tok_seq, T,
                            nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, split_keys, max_splits,
-                           scratch, out_f32, keep_first, softcap, sink_vals, stream);
+                           scratch, out_f32, keep_first, softcap, sink_vals, dist, dist_len, stream);
   if (dtype == DT_BF16)
     return dispatch<__nv_bfloat16>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos,
                                    tok_seq, T, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale,
-                                   split_keys, max_splits, scratch, out_f32, keep_first, softcap, sink_vals, stream);
+                                   split_keys, max_splits, scratch, out_f32, keep_first, softcap, sink_vals,
+                                   dist, dist_len, stream);
   set_error("attn_tokens: unsupported element type %d", dtype);
   return ERR_UNSUPPORTED;
 }
@@ -511,7 +526,7 @@ extern "C" int exl3_attn_tokens_wide(const void* q, int64_t q_row_stride, void* 
                                      cudaStream_t stream) {
   return exl3_attn_tokens_opt(q, q_row_stride, out, out_f32, dtype, k_pool, v_pool, block_table, bt_stride, tok_pos, tok_seq,
                               T, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, split_keys, max_splits,
-                              scratch, scratch_bytes, 0, 0.0f, nullptr, stream);
+                              scratch, scratch_bytes, 0, 0.0f, nullptr, nullptr, 0, stream);
 }
 
 extern "C" int exl3_attn_tokens_ex(const void* q, int64_t q_row_stride, void* out, int dtype,

@@ -154,6 +154,14 @@ __device__ inline void rope_sincos(float p, float hi, float lo, float* sn, float
   *cs = fmaf(c, cd, -s * sd);
 }
 
+// Score biases by distance, one table per query head: row h of the table holds DIST_PAD zeros, the biases for keys 0, 1,
+// ... len - 1 positions back, and DIST_PAD zeros, so that a kernel that walks a tile of queries over a tile of keys may
+// read a little outside of 0 .. len - 1 without looking.
+constexpr int DIST_PAD = 128;
+__host__ __device__ inline const float* dist_row(const float* table, int len, int head) {
+  return table + (int64_t)head * (len + 2 * DIST_PAD) + DIST_PAD;
+}
+
 template <typename... KArgs, typename... Args>
 inline void launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
                        Args&&... args) {

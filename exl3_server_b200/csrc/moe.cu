@@ -4,7 +4,9 @@
 //   router   z = Wr x (float32), s = softmax(z) or sigmoid(z) over all router outputs, choice c = s + correction;
 //            the outputs form equal groups of neighbours, a group's score is its largest c, only the outputs of the
 //            `keep` best groups can be chosen; the `top` largest c among those are the token's picks, each with the
-//            weight s * scale (no renormalisation).  One more row of Wr may follow the router's: its sigmoid is a
+//            weight s * scale (no renormalisation).  A third kind of score ("picked"): correction is a bias of the
+//            logits, the choice is made by z + bias and the weights are the softmax over the chosen logits alone, times
+//            scale.  One more row of Wr may follow the router's: its sigmoid is a
 //            gate per token (for a shared expert) that the same kernel leaves beside the picks.
 //   plan     the pairs (token, pick) whose pick is an expert with weights, ordered by expert and cut into tiles of
 //            at most a given number of rows of one expert; everything stays on the device (no count reaches the host), so the
@@ -51,11 +53,14 @@ __device__ inline void route_choice(int t, int lane, float* zt, float* ct, float
                                     const float* __restrict__ corr, int E, int S, int groups, int keep, int top,
                                     float scale, int score_kind, int* idx, float* wt, float* gate_out) {
   // score_kind: bit 0 set: sigmoid scores (else softmax); bit 1 set: a group's score is the sum of its two largest
-  // choice scores (else its largest)
-  const bool group_pair = (score_kind & 2) != 0;
+  // choice scores (else its largest); bit 2 set: the choice is by the biased logits and the weights are the softmax over
+  // the chosen ones
+  const bool group_pair = (score_kind & 2) != 0, picked = (score_kind & 4) != 0;
   score_kind &= 1;
   if (S && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-zt[E]));
-  if (score_kind == 0) {
+  if (picked) {
+    for (int e = lane; e < E; e += 32) ct[e] = zt[e] + corr[e];
+  } else if (score_kind == 0) {
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, zt[e]);
     mx = warp_max(mx);
@@ -104,6 +109,7 @@ __device__ inline void route_choice(int t, int lane, float* zt, float* ct, float
       if (gkt[e / per] == 0.0f) ct[e] = -INFINITY;   // not 0: choice scores may be negative
     __syncwarp();
   }
+  float best = 0.0f, sum = 0.0f;                     // of a choice by logits: the largest, and the weights' sum (lane 0)
   for (int r = 0; r < top; ++r) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -113,7 +119,14 @@ __device__ inline void route_choice(int t, int lane, float* zt, float* ct, float
     if (lane == 0) {
       if (bi < E) {
         idx[(int64_t)t * top + r] = bi;
-        wt[(int64_t)t * top + r] = zt[bi] * scale;
+        if (picked) {
+          if (r == 0) best = bv;
+          const float w = expf(bv - best);
+          sum += w;
+          wt[(int64_t)t * top + r] = w;
+        } else {
+          wt[(int64_t)t * top + r] = zt[bi] * scale;
+        }
         ct[bi] = -INFINITY;
       } else {
         idx[(int64_t)t * top + r] = -1;
@@ -121,6 +134,9 @@ __device__ inline void route_choice(int t, int lane, float* zt, float* ct, float
       }
     }
     __syncwarp();
+  }
+  if (picked && lane == 0) {
+    for (int r = 0; r < top; ++r) wt[(int64_t)t * top + r] = wt[(int64_t)t * top + r] / sum * scale;
   }
 }
 
@@ -285,6 +301,7 @@ __device__ inline float moe_act(float v, int act) {
   if (act == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
   if (act == 2) return 0.5f * v * (1.0f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
   if (act == 3) return v / (1.0f + expf(-v));
+  if (act == 4) { const float r = fmaxf(v, 0.0f); return r * r; }
   return v;
 }
 
@@ -446,6 +463,77 @@ moe_gather_kernel(const __nv_bfloat16* x, int64_t ldx, int top, const int* order
   for (int c = threadIdx.x; c < K / 8; c += blockDim.x) dst[c] = __ldcg(src + c);
 }
 
+// The weighted sum and the norm on it with the residual's step, in one kernel (a block a token): v = sum_k weight[t, k]
+// y[t, k] + gate[t] shared[t], h[t] += v / sqrt(mean(v^2) + eps) * w, x[t] = h[t] in x's type.  A thread keeps its pieces
+// of four values in registers: rows of up to CN_THREADS * 4 * CN_VECS values, a multiple of 4.  No identity picks.
+constexpr int CN_THREADS = 256, CN_VECS = 8;
+
+__device__ inline void cn_load4(const float* p, float (&v)[4]) { load_vec_cg(p, v); }
+__device__ inline void cn_load4(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 r = __ldcg(reinterpret_cast<const uint2*>(p));
+  v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+  v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+}
+
+template <typename TS>
+__global__ void __launch_bounds__(CN_THREADS)
+moe_combine_norm_kernel(const float* y, const int* idx, const float* wt, const TS* shared, const float* gate, float* h,
+                        const float* __restrict__ w, float eps, __nv_bfloat16* x, int H, int top, int n_experts) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const int64_t base = (int64_t)t * H;
+  float v[CN_VECS][4];
+  float ss = 0.0f;
+  const float gt = gate ? __ldcg(gate + t) : 1.0f;
+#pragma unroll
+  for (int p = 0; p < CN_VECS; ++p) {
+    const int c = (p * CN_THREADS + threadIdx.x) * 4;
+    if (c < H) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[p][e] = 0.0f;
+      for (int k = 0; k < top; ++k) {
+        const int ex = __ldcg(idx + (int64_t)t * top + k);
+        if (ex < 0 || ex >= n_experts) continue;
+        const float wk = __ldcg(wt + (int64_t)t * top + k);
+        float a[4];
+        load_vec_cg(y + ((int64_t)t * top + k) * H + c, a);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[p][e] = fmaf(wk, a[e], v[p][e]);
+      }
+      if (shared) {
+        float a[4];
+        cn_load4(shared + base + c, a);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[p][e] = fmaf(gt, a[e], v[p][e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss += v[p][e] * v[p][e];
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)H + eps);
+#pragma unroll
+  for (int p = 0; p < CN_VECS; ++p) {
+    const int c = (p * CN_THREADS + threadIdx.x) * 4;
+    if (c < H) {
+      float a[4], wv[4];
+      load_vec_cg(h + base + c, a);
+      load_vec(w + c, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a[e] += v[p][e] * inv * wv[e];
+      store_vec(h + base + c, a);
+      if (x) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
+        uint2 r;
+        r.x = *reinterpret_cast<uint32_t*>(&lo);
+        r.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(x + base + c) = r;
+      }
+    }
+  }
+}
+
 // VEC columns a thread (4: H a multiple of 4, float4 loads of y and stores of out).
 template <typename TX, int VEC>
 __global__ void __launch_bounds__(256)
@@ -505,7 +593,7 @@ extern "C" int exl3_moe_route(const void* x, int x_dtype, int64_t ldx, const flo
                               float* wt, float* gate_out, cudaStream_t stream) {
   if (T == 0) return 0;
   if (T < 0 || W < 1 || E < 1 || extra < 0 || extra > 1 || groups < 1 || E % groups != 0 || keep < 1 || keep > groups ||
-      top < 1 || top > keep * (E / groups) || (extra && gate_out == nullptr) || score_kind < 0 || score_kind > 3) {
+      top < 1 || top > keep * (E / groups) || (extra && gate_out == nullptr) || score_kind < 0 || score_kind > 7) {
     set_error("moe_route: bad sizes T=%d width=%d outputs=%d groups=%d keep=%d top=%d", T, W, E, groups, keep, top);
     return ERR_BAD_ARGUMENT;
   }
@@ -581,7 +669,7 @@ extern "C" int exl3_moe_gemm(const void* A, int a_dtype, int64_t lda, int a_div,
                              const int* order, const int* plan, void* out, int out_dtype, int P, int n_experts, int N,
                              int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || N < 1 || K < 1 || a_div < 1 || act < 0 || act > 3) {
+  if (P < 0 || n_experts < 1 || N < 1 || K < 1 || a_div < 1 || act < 0 || act > 4) {
     set_error("moe_gemm: bad sizes pairs=%d experts=%d N=%d K=%d", P, n_experts, N, K);
     return ERR_BAD_ARGUMENT;
   }
@@ -606,7 +694,7 @@ extern "C" int exl3_moe_gemv_rows() { return MV_ROWS; }
 extern "C" int exl3_moe_gemv(const void* A, int64_t lda, int a_div, const void* W, const int* order, const int* plan,
                              void* out, int out_dtype, int P, int n_experts, int N, int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || N < 1 || K < 8 || K % 8 != 0 || lda % 8 != 0 || a_div < 1 || act < 0 || act > 3 ||
+  if (P < 0 || n_experts < 1 || N < 1 || K < 8 || K % 8 != 0 || lda % 8 != 0 || a_div < 1 || act < 0 || act > 4 ||
       !aligned16(A) || !aligned16(W)) {
     set_error("moe_gemv: bad sizes pairs=%d experts=%d N=%d K=%d (K and the row pitch multiples of 8, 16-byte aligned)", P,
               n_experts, N, K);
@@ -654,6 +742,26 @@ extern "C" int exl3_moe_combine(const float* y, const int* idx, const float* wt,
   else { if (vec) EXL3_COMBINE(__nv_bfloat16, 4); else EXL3_COMBINE(__nv_bfloat16, 1); }
 #undef EXL3_COMBINE
   return launch_status("moe_combine");
+}
+
+extern "C" int exl3_moe_combine_norm(const float* y, const int* idx, const float* wt, const void* shared, int shared_dtype,
+                                     const float* gate, float* h, const float* w, float eps, void* x, int T, int H, int top,
+                                     int n_experts, cudaStream_t stream) {
+  if (T == 0) return 0;
+  if (T < 0 || H < 4 || H % 4 != 0 || H > CN_THREADS * 4 * CN_VECS || top < 1 || y == nullptr || h == nullptr || w == nullptr ||
+      !aligned16(y) || !aligned16(h) || !aligned16(w) || !aligned16(shared) || !aligned16(x)) {
+    set_error("moe_combine_norm: bad sizes rows=%d width=%d (a multiple of 4, at most %d, 16-byte aligned)", T, H,
+              CN_THREADS * 4 * CN_VECS);
+    return ERR_BAD_ARGUMENT;
+  }
+  if (shared_dtype == DT_F32)
+    launch_pdl(moe_combine_norm_kernel<float>, dim3(T), dim3(CN_THREADS), 0, stream, y, idx, wt, static_cast<const float*>(shared),
+               gate, h, w, eps, static_cast<__nv_bfloat16*>(x), H, top, n_experts);
+  else if (shared_dtype == DT_BF16)
+    launch_pdl(moe_combine_norm_kernel<__nv_bfloat16>, dim3(T), dim3(CN_THREADS), 0, stream, y, idx, wt,
+               static_cast<const __nv_bfloat16*>(shared), gate, h, w, eps, static_cast<__nv_bfloat16*>(x), H, top, n_experts);
+  else { set_error("moe_combine_norm: unsupported element type %d", shared_dtype); return ERR_UNSUPPORTED; }
+  return launch_status("moe_combine_norm");
 }
 
 // The activation of experts with a bounded gate: rows of gu hold [gate (I) | up (I)];

@@ -42,6 +42,7 @@ __device__ inline float mt_act(float v, int act) {
   if (act == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
   if (act == 2) return 0.5f * v * (1.0f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
   if (act == 3) return v / (1.0f + expf(-v));
+  if (act == 4) { const float r = fmaxf(v, 0.0f); return r * r; }
   return v;
 }
 
@@ -214,7 +215,7 @@ extern "C" int exl3_moe_tc_supported(int N, int K) { return N >= 8 && N % 8 == 0
 extern "C" int exl3_moe_gemm_tc(const void* A, const void* W, const int* order, const int* plan, void* out, int out_dtype,
                                 int P, int n_experts, int N, int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || !exl3_moe_tc_supported(N, K) || act < 0 || act > 3 ||
+  if (P < 0 || n_experts < 1 || !exl3_moe_tc_supported(N, K) || act < 0 || act > 4 ||
       (out_dtype != DT_BF16 && out_dtype != DT_F32)) {
     set_error("moe_gemm_tc: needs N and K multiples of 8 and a bfloat16 or float32 output, got pairs=%d experts=%d N=%d "
               "K=%d out=%d", P, n_experts, N, K, out_dtype);

@@ -522,16 +522,18 @@ def attn_tokens_ex(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool
                    T: int, heads: int, kv_heads: int, head_dim: int, value_dim: int, page: int, window: int,
                    chunk: int, sink: bool, scale: float, split_keys: int, max_splits: int,
                    scratch: Optional[torch.Tensor], keep_first: int = 0, softcap: float = 0.0,
-                   sink_vals: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``attn_tokens`` in its general form: rows of the key pool hold ``head_dim`` features and rows of the value
     pool ``value_dim`` (each pool's last dimension is its row pitch; multiples of 8; values may be wider than keys);
     ``chunk`` > 0 also hides every key before ``floor(pos / chunk) * chunk``; ``sink`` adds one to the softmax's
     denominator (``sink_vals`` float32 ``[heads]``: ``exp`` of a score per head instead of one).  With a window,
     keys at positions below ``keep_first`` stay visible (``max_splits`` then counts their chunks too); ``softcap``
-    > 0 caps the scaled scores, ``c tanh(s / c)``.  ``out`` is ``[T, heads, value_dim]`` in the cache's type or
+    > 0 caps the scaled scores, ``c tanh(s / c)``; ``dist`` (a ``distance_table``) adds a bias per head and distance to
+    them.  ``out`` is ``[T, heads, value_dim]`` in the cache's type or
     float32 (for callers that go on in float32) and the scratch is sized with ``value_dim``."""
     if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
         raise KernelLibraryError("attn_tokens_ex: sink scores must be float32 [heads], with the sink on")
+    dist_len = _distance_len(dist, heads, "attn_tokens_ex")
     if k_pool.dtype != q.dtype or v_pool.dtype != q.dtype or out.dtype not in (q.dtype, torch.float32):
         raise KernelLibraryError("attn_tokens_ex: q, cache and out differ in element type")
     nbytes = 0 if scratch is None else scratch.numel() * scratch.element_size()
@@ -542,8 +544,49 @@ def attn_tokens_ex(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool
         _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim), _c_int(k_pool.shape[-1]),
         _c_int(v_pool.shape[-1]), _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0),
         _c_float(scale), _c_int(split_keys), _c_int(max_splits), _ptr(scratch), _c_size_t(nbytes), _c_int(keep_first),
-        _c_float(softcap), _ptr(sink_vals), _stream()), "attn_tokens_ex")
+        _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()), "attn_tokens_ex")
     return out
+
+
+DIST_PAD = 128       # zeros around a row of distance biases (common.cuh)
+
+
+def distance_table(biases: torch.Tensor) -> torch.Tensor:
+    """Score biases ``[heads, n]`` for keys 0 .. n - 1 positions back (nothing is added further back) as the attention
+    kernels take them: float32 rows with ``DIST_PAD`` zeros on both sides."""
+    return torch.nn.functional.pad(biases.to(torch.float32), (DIST_PAD, DIST_PAD)).contiguous()
+
+
+def _distance_len(dist: Optional[torch.Tensor], heads: int, what: str) -> int:
+    if dist is None:
+        return 0
+    if dist.dtype != torch.float32 or dist.dim() != 2 or dist.shape[0] != heads or dist.shape[1] < 2 * DIST_PAD or \
+            not dist.is_contiguous():
+        raise KernelLibraryError(f"{what}: distance biases must be a contiguous float32 distance_table with a row per head")
+    return dist.shape[1] - 2 * DIST_PAD
+
+
+def embed_sinusoid(ids: torch.Tensor, tok_pos: torch.Tensor, table: torch.Tensor, scale: float, frequencies: torch.Tensor,
+                   norm_w: Optional[torch.Tensor], eps: float, x_dtype: Optional[torch.dtype]):
+    """``table[id] * scale`` plus a sinusoidal vector of the token's position (``frequencies``: a ``rotary_table`` of
+    ``ceil(H / 2)``), then an RMS norm when ``norm_w`` (float32) is given (see sinusoid_embed.cu).  Returns ``(h float32
+    [T, H], the same in bfloat16 when x_dtype is bfloat16, else None)``."""
+    T = ids.numel()
+    V, H = table.shape
+    _contig(table, "table")
+    if ids.dtype != torch.int32 or tok_pos.dtype != torch.int32 or tok_pos.numel() < T:
+        raise KernelLibraryError("embed_sinusoid: ids and positions must be int32, one position a token")
+    if frequencies.dtype != torch.float32 or tuple(frequencies.shape) != (2, (H + 1) // 2) or not frequencies.is_contiguous():
+        raise KernelLibraryError("embed_sinusoid: frequencies must be a rotary_table of ceil(H / 2)")
+    if norm_w is not None and (norm_w.dtype != torch.float32 or norm_w.numel() != H):
+        raise KernelLibraryError("embed_sinusoid: the norm's weight must be float32 [H]")
+    h = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    x = torch.empty((T, H), dtype=torch.bfloat16, device=table.device) if x_dtype == torch.bfloat16 else None
+    _check(library().exl3_embed_sinusoid(
+        _ptr(ids), _ptr(tok_pos), _ptr(table), _c_int(dtype_code(table.dtype)), _c_float(scale), _ptr(frequencies[0]),
+        _ptr(frequencies[1]), _ptr(norm_w), _c_float(eps), _ptr(h), _ptr(x), _c_int(T), _c_int(H), _c_int(V), _stream()),
+        "embed_sinusoid")
+    return h, x
 
 
 def embed_hashed(ids: torch.Tensor, tok_pos: torch.Tensor, tok_seq: torch.Tensor, row_start: torch.Tensor,
@@ -574,18 +617,19 @@ def qk_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_
             mscale: float, k_mul: float, mix: Optional[tuple], tok_pos: torch.Tensor, tok_seq: torch.Tensor,
             block_table: Optional[torch.Tensor], page: int, q_dtype: torch.dtype,
             k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
-            k_dtype: Optional[torch.dtype] = None):
+            k_dtype: Optional[torch.dtype] = None, temperature: Optional[tuple] = None):
     """Norm, rotation, value mixing and the cache write between an attention's joint projection ``x [T, ld]`` and
     the attention (see qk_prep.cu).  ``mix``: ``(lambda tensor, v_src [T, *] view)`` or None.  Returns ``(q, k)``:
     the queries ``[T, heads * head_pad]`` and, when there is no ``k_pool``, the keys ``[T, kv_heads * head_pad]``
-    (else None)."""
+    (else None).  ``kv_heads`` 0: queries only (``v_off`` -1, no pools).  ``temperature``: ``(coef, every)``; queries at
+    position p are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
     T = x.shape[0]
     if x.stride(1) != 1:
         raise KernelLibraryError("qk_prep: rows of x must be dense")
     hi, lo = (_rotary_rows(inv_freq, rot, "qk_prep") if rot else (_c_void_p(0), _c_void_p(0)))
     q = torch.empty((T, heads * head_pad), dtype=q_dtype, device=x.device)
     k = None
-    if k_pool is None:
+    if k_pool is None and kv_heads > 0:
         k = torch.empty((T, kv_heads * head_pad), dtype=k_dtype or q_dtype, device=x.device)
     lam, v_src = mix if mix is not None else (None, None)
     if v_src is not None and v_src.stride(1) != 1:
@@ -600,7 +644,9 @@ def qk_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_
         _c_int64(v_src.stride(0) if v_src is not None else 0), _ptr(tok_pos), _ptr(tok_seq), _ptr(block_table),
         _c_int(block_table.stride(0) if block_table is not None else 0), _c_int(page), _ptr(q),
         _c_int(dtype_code(q.dtype)), _ptr(k), _c_int(dtype_code(k.dtype) if k is not None else 0), _ptr(k_pool),
-        _ptr(v_pool), _c_int(dtype_code(k_pool.dtype) if k_pool is not None else 0), _stream()), "qk_prep")
+        _ptr(v_pool), _c_int(dtype_code(k_pool.dtype) if k_pool is not None else 0),
+        _c_float(temperature[0] if temperature else 0.0), _c_float(temperature[1] if temperature else 0.0), _stream()),
+        "qk_prep")
     return q, k
 
 
@@ -909,13 +955,14 @@ def attn_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
                     tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, heads: int, kv_heads: int,
                     head_dim: int, page: int, window: int, scale: float, variant: int = 0, chunk: int = 0,
                     sink: bool = False, keep_first: int = 0, softcap: float = 0.0,
-                    sink_vals: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of whole prompts on tcgen05 tensor cores (tiles of 128 queries; see
     attention_prefill_tc.cu).  ``k_pool`` / ``v_pool``: one layer's ``[pages, kv_heads, 64, head_dim]``.
     ``variant``: 0 lets the kernel choose by the number of blocks between a tile a block, four blocks per SM (heads
     of 64) and two tiles a block (the list's first with its last, and so on: list the tiles with the most keys
     to visit first); 1, 2 and 3 force one of them (the same numbers every way).  ``chunk``, ``sink``, ``keep_first``,
-    ``softcap`` and ``sink_vals`` as in ``attn_tokens_ex``."""
+    ``softcap``, ``sink_vals`` and ``dist`` as in ``attn_tokens_ex``."""
+    dist_len = _distance_len(dist, heads, "attn_prefill_tc")
     if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
         raise KernelLibraryError("attn_prefill_tc: sink scores must be float32 [heads], with the sink on")
     if k_pool.dtype != q.dtype or v_pool.dtype != q.dtype or out.dtype != q.dtype:
@@ -928,7 +975,8 @@ def attn_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
         _c_int64(pool_rows), _ptr(block_table), _c_int(block_table.stride(0)), _ptr(row_start), _ptr(row_pos0),
         _ptr(tile_seq), _ptr(tile_q0), _c_int(n_tiles), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
         _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0), _c_float(scale), _c_int(variant),
-        _c_int(keep_first), _c_float(softcap), _ptr(sink_vals), _stream()), "attn_prefill_tc")
+        _c_int(keep_first), _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()),
+        "attn_prefill_tc")
     return out
 
 
@@ -964,7 +1012,8 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
                 kv_heads: int, head_dim: int, page: int, window: int, scale: float, split_keys: int,
                 max_splits: int, scratch: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor] = None,
                 rot: int = 0, pos_scale: float = 1.0, write_new: bool = False, head_split: int = 1,
-                in_block: int = 0, twins: int = 1, chunk: int = 0, sink: bool = False) -> torch.Tensor:
+                in_block: int = 0, twins: int = 1, chunk: int = 0, sink: bool = False,
+                sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of T query tokens over the paged cache on the tensor cores (see attention_decode.cu);
     arguments and scratch as ``attn_tokens``.  With ``write_new``, ``q`` is the fused q|k|v output of the
     projection, every token is its sequence's only new one and the cache holds the positions before it: the
@@ -977,8 +1026,11 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
     chunks; the first block merges and reads the second one's records out of its shared memory): no scratch, no
     tickets; results differ from the other way's by rounding (another order of the same sums).  ``twins`` 2 (with
     ``in_block`` 1 or 2, an even ``head_split`` and groups of up to 8 heads): a block takes two groups of query heads
-    of a kv head, whose warps walk the same pages out of the same rings; changes no result.  ``chunk`` and ``sink`` as
-    in ``attn_tokens_ex``."""
+    of a kv head, whose warps walk the same pages out of the same rings; changes no result.  ``chunk``, ``sink``,
+    ``sink_vals`` and ``dist`` as in ``attn_tokens_ex``."""
+    if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
+        raise KernelLibraryError("attn_decode: sink scores must be float32 [heads], with the sink on")
+    dist_len = _distance_len(dist, heads, "attn_decode")
     if k_pool.dtype != q.dtype or v_pool.dtype != q.dtype or out.dtype != q.dtype:
         raise KernelLibraryError("attn_decode: q, cache and out differ in element type")
     _contig(k_pool, "k_pool")
@@ -996,7 +1048,7 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
         _c_int(kv_heads), _c_int(head_dim), _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0),
         _c_float(scale), _c_int(split_keys), _c_int(max_splits), _ptr(scratch), _c_size_t(nbytes), hi, lo, _c_int(rot),
         _c_float(pos_scale), _c_int(1 if write_new else 0), _c_int(head_split), _c_int(int(in_block)),
-        _c_int(int(twins)), _stream()), "attn_decode")
+        _c_int(int(twins)), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()), "attn_decode")
     return out
 
 
@@ -1124,8 +1176,8 @@ def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     return x
 
 
-MOE_ACTIVATIONS = {"none": 0, "gelu": 1, "gelu_tanh": 2, "silu": 3}
-MOE_SCORES = {"softmax": 0, "sigmoid": 1}
+MOE_ACTIVATIONS = {"none": 0, "gelu": 1, "gelu_tanh": 2, "silu": 3, "relu2": 4}
+MOE_SCORES = {"softmax": 0, "sigmoid": 1, "picked": 4}
 MOE_GROUP_SCORES = {"max": 0, "top2": 2}     # added to the score's code
 
 
@@ -1152,7 +1204,8 @@ def moe_tc_status() -> int:
 def moe_route(x: torch.Tensor, wr: torch.Tensor, corr: torch.Tensor, outputs: int, extra: int, groups: int, keep: int,
               top: int, scale: float, score: str = "softmax", group_score: str = "max"):
     """The router of a routed feed-forward (see moe.cu): ``wr`` float32 ``[outputs + extra, W]``, ``corr`` float32
-    ``[outputs]`` added to the scores for the choice only.  Returns ``(idx int32 [T, top], weight float32 [T, top],
+    ``[outputs]`` added to the scores for the choice only (``score`` ``"picked"``: added to the logits, by which the choice
+    is then made; the weights are the softmax over the chosen logits alone).  Returns ``(idx int32 [T, top], weight float32 [T, top],
     gate float32 [T] or None)``: the gate is the sigmoid of the extra row's product.  ``group_score``: a group's
     score is its largest choice score (``max``) or the sum of its two largest (``top2``)."""
     T, W = x.shape
@@ -1272,6 +1325,34 @@ def moe_combine(y: Optional[torch.Tensor], idx: torch.Tensor, wt: torch.Tensor, 
         _c_int(dtype_code(shared.dtype) if shared is not None else 0), _ptr(gate), _ptr(out), _c_int(T), _c_int(H),
         _c_int(top), _c_int(n_experts), _stream()), "moe_combine")
     return out
+
+
+def moe_combine_norm_supported(width: int) -> bool:
+    return width % 4 == 0 and width <= 8192
+
+
+def moe_combine_norm(y: torch.Tensor, idx: torch.Tensor, wt: torch.Tensor, shared: Optional[torch.Tensor],
+                     gate: Optional[torch.Tensor], n_experts: int, h: torch.Tensor, weight: torch.Tensor, eps: float,
+                     want_x: bool) -> Optional[torch.Tensor]:
+    """``moe_combine`` (no identity picks) and ``norm_add`` in one kernel: with ``v`` the weighted sum, ``h += v *
+    rsqrt(mean(v^2) + eps) * weight`` in place (float32); returns the new ``h`` in bfloat16 with ``want_x``."""
+    T, top = idx.shape
+    H = h.shape[1]
+    if h.dtype != torch.float32 or y.dtype != torch.float32 or weight.dtype != torch.float32 or weight.numel() != H or \
+            tuple(y.shape) != (T * top, H) or h.shape[0] != T:
+        raise KernelLibraryError("moe_combine_norm: h [T, H], y [T * top, H] and the weight [H] must be float32")
+    for t, name in ((h, "h"), (y, "y"), (weight, "weight")):
+        _contig(t, name)
+    if shared is not None:
+        _contig(shared, "shared")
+        if tuple(shared.shape) != (T, H):
+            raise KernelLibraryError(f"moe_combine_norm: shared is {tuple(shared.shape)}, h is {tuple(h.shape)}")
+    x = torch.empty((T, H), dtype=torch.bfloat16, device=h.device) if want_x else None
+    _check(library().exl3_moe_combine_norm(
+        _ptr(y), _ptr(idx), _ptr(wt), _ptr(shared), _c_int(dtype_code(shared.dtype) if shared is not None else 0), _ptr(gate),
+        _ptr(h), _ptr(weight), _c_float(eps), _ptr(x), _c_int(T), _c_int(H), _c_int(top), _c_int(n_experts), _stream()),
+        "moe_combine_norm")
+    return x
 
 
 def maps_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, maps: int, d: int,

@@ -97,7 +97,9 @@ class OutNormBlock:
         x = stream.act if stream.act is not None and stream.pending is None else self.mixer_norm.add_normed(stream, None)
         x = self.mixer_norm.add_normed(stream, self.mixer.forward(x, batch, kv, state))
         if self.feed_forward is not None:
-            self.feed_forward_norm.add_normed(stream, self.feed_forward.forward(x, batch))
+            # a routed feed-forward hands over the pieces of its weighted sum: the sum is then part of the norm's kernel
+            run = getattr(self.feed_forward, "forward_pieces", self.feed_forward.forward)
+            self.feed_forward_norm.add_normed(stream, run(x, batch))
 
     def weight_bytes(self) -> int:
         return sum(p.weight_bytes() for p in (self.mixer, self.feed_forward, self.mixer_norm, self.feed_forward_norm)

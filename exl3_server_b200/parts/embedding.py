@@ -21,6 +21,7 @@ from ..ops import kernels as K
 from ..weights.loader import TensorSpec
 from .base import BuildContext, ResidualStream, StateRequest
 from .linear import Linear
+from .norm import RMSNorm
 from .registry import register_embedding, register_head
 from .spec import EmbeddingSpec, HeadSpec
 
@@ -110,6 +111,47 @@ class HashedPairEmbedding:
         return (self.table.numel() + self.pairs.numel()) * self.table.element_size()
 
 
+class SinusoidEmbedding:
+    """``h0[t] = norm(E[id_t] * scale + P[p_t])``: the token's row plus a sinusoidal vector of its position, entry 2i
+    ``sin(p base^(-2i / width))`` and entry 2i + 1 the cosine, then an RMS norm where the spec has one.  One kernel, float32
+    inside; in the bfloat16 path it also leaves the row in 16 bits for the first layer.  Parameters of the spec: ``base``,
+    ``norm`` (a ``NormSpec`` of kind ``rms``, or None) and ``norm_name``."""
+
+    takes_batch = True
+
+    @staticmethod
+    def tensor_specs(spec: EmbeddingSpec) -> List[TensorSpec]:
+        out = [TensorSpec(spec.name, (spec.vocab, spec.width))]
+        if spec.params.get("norm") is not None:
+            out += RMSNorm.tensor_specs(spec.params["norm"], spec.params["norm_name"])
+        return out
+
+    def __init__(self, spec: EmbeddingSpec, tensors: Dict[str, torch.Tensor], ctx: BuildContext):
+        self.spec, self.dtype = spec, ctx.dtype
+        self.table = tensors[spec.name].to(ctx.dtype).contiguous()
+        i = torch.arange((spec.width + 1) // 2, dtype=torch.float64)
+        base = torch.tensor(float(spec.params.get("base", 10000.0)), dtype=torch.float64)
+        self.frequencies = K.rotary_table(torch.pow(base, -2.0 * i / spec.width)).to(ctx.device)
+        self.norm_w, self.eps = None, 0.0
+        norm = spec.params.get("norm")
+        if norm is not None:
+            if norm.kind != "rms":
+                raise ValueError(f"sinusoid embedding: the norm must be of kind 'rms', got {norm.kind!r}")
+            self.norm_w = RMSNorm(norm, tensors, spec.params["norm_name"], ctx).weight.float().contiguous()
+            self.eps = norm.eps
+
+    def forward(self, token_ids: torch.Tensor, batch, state: Optional[torch.Tensor]) -> ResidualStream:
+        h, x = K.embed_sinusoid(token_ids, batch.tok_pos, self.table, float(self.spec.scale), self.frequencies, self.norm_w,
+                                self.eps, self.dtype)
+        stream = ResidualStream(h)
+        stream.act = x if x is not None else h
+        return stream
+
+    def weight_bytes(self) -> int:
+        return self.table.numel() * self.table.element_size()
+
+
 register_embedding("table", Embedding)
+register_embedding("table_sinusoid", SinusoidEmbedding)
 register_embedding("table_hashed_pair", HashedPairEmbedding)
 register_head("linear", Head)

@@ -10,8 +10,12 @@ outputs have no tensors and stand for the input ``r`` itself.  The output is the
 the spec has ``shared_inner``, a shared expert of the same form (``shared.up``, ``shared.down``) that every token
 runs, times ``sigmoid(w_sg . r)`` (``shared.sg``, one number per token).
 
+Variants: with ``score`` ``"picked"`` the choice is made by the logits themselves and a pick's weight is the softmax over
+the chosen logits alone, times ``scale``; ``router_bias`` (with ``"picked"`` only) adds a stored bias ``router.b`` to the
+logits.  ``correction`` False: there is no correction.  ``shared_gate`` False: the shared expert is added as it is.
+
 Parameters of the spec: ``experts``, ``identity``, ``top``, ``scale``, ``groups``, ``keep``, ``activation`` (``gelu``,
-``gelu_tanh`` or ``silu``), ``score`` (``softmax`` or ``sigmoid``), ``group_score`` (``max``, or ``top2``: a group's
+``gelu_tanh``, ``silu`` or ``relu2``), ``score`` (``softmax``, ``sigmoid`` or ``picked``), ``group_score`` (``max``, or ``top2``: a group's
 score is the sum of its two largest choice scores), ``shared_inner`` (0: none); ``inner`` is an expert's hidden size.
 ``expert`` = ``"clamped_glu"`` makes the experts (and the shared one) gated with a bounded gate, ``Wd (g sigmoid(alpha
 g) (u + 1))``, ``g = min(Wg r, limit)``, ``u = clamp(Wu r, -limit, limit)`` (tensors ``e<i>.gate``, ``e<i>.up``,
@@ -23,7 +27,8 @@ How it runs (``csrc/moe.cu``): the router kernel also computes the shared expert
 of the router's float32 matrix); a one-block kernel orders the step's (token, pick) pairs by expert into tiles, on the
 device, so a step is the same list of launches whatever the router chose (it can be part of a recorded graph); the
 experts' weights are stacked ``[experts, out, in]`` and both projections are grouped products over the tiles; the
-last kernel sums picks, identity picks and the gated shared expert in float32.  Which product runs depends on the
+last kernel sums picks, identity picks and the gated shared expert in float32 (an arrangement that norms this part's output
+asks for the pieces, ``forward_pieces``, and gets sum, norm and residual step from one kernel).  Which product runs depends on the
 step only through its number of pairs: in bfloat16, few pairs (decode) take the kernel that reads each expert's
 matrix once with a warp per output feature, many pairs (prompts) are gathered into the plan's order and go through
 the tcgen05 grouped product; float32, and sizes those two do not take, use the CUDA-core tiles.
@@ -44,6 +49,16 @@ from .spec import FeedForwardSpec
 
 FEW_PAIRS = 128       # up to here the few-row product; from MANY_PAIRS on the tensor cores
 MANY_PAIRS = 512
+
+
+class PickedSum:
+    """``sum_k wt[t, k] y[t, k] + gate[t] shared[t]``, not summed yet."""
+
+    def __init__(self, y, idx, wt, shared, gate, n_experts: int):
+        self.y, self.idx, self.wt, self.shared, self.gate, self.n_experts = y, idx, wt, shared, gate, n_experts
+
+    def norm_add(self, h: torch.Tensor, weight: torch.Tensor, eps: float, want_x: bool):
+        return K.moe_combine_norm(self.y, self.idx, self.wt, self.shared, self.gate, self.n_experts, h, weight, eps, want_x)
 
 
 class RoutedFeedForward:
@@ -72,7 +87,11 @@ class RoutedFeedForward:
     @classmethod
     def tensor_specs(cls, spec: FeedForwardSpec, prefix: str) -> List[TensorSpec]:
         E, I, shared = cls._sizes(spec)
-        out = [TensorSpec(prefix + "router", (E + I, spec.width)), TensorSpec(prefix + "correction", (E + I,))]
+        out = [TensorSpec(prefix + "router", (E + I, spec.width))]
+        if spec.params.get("correction", True):
+            out.append(TensorSpec(prefix + "correction", (E + I,)))
+        if spec.params.get("router_bias", False):
+            out.append(TensorSpec(prefix + "router.b", (E + I,)))
         for e in range(E):
             if cls._clamped(spec):
                 out.append(TensorSpec(f"{prefix}e{e}.gate", (spec.inner, spec.width)))
@@ -80,7 +99,8 @@ class RoutedFeedForward:
                     TensorSpec(f"{prefix}e{e}.down", (spec.width, spec.inner))]
         if shared:
             out += cls._shared_class(spec).tensor_specs(cls._shared_spec(spec, shared), prefix + "shared.")
-            out.append(TensorSpec(prefix + "shared.sg", (1, spec.width)))
+            if spec.params.get("shared_gate", True):
+                out.append(TensorSpec(prefix + "shared.sg", (1, spec.width)))
         return out
 
     def __init__(self, spec: FeedForwardSpec, tensors: Dict[str, torch.Tensor], prefix: str, ctx: BuildContext):
@@ -107,9 +127,18 @@ class RoutedFeedForward:
         self.shared = None
         if shared:
             self.shared = self._shared_class(spec)(self._shared_spec(spec, shared), tensors, prefix + "shared.", ctx)
-            rows.append(tensors[prefix + "shared.sg"].float().reshape(1, spec.width))
+            if p.get("shared_gate", True):
+                rows.append(tensors[prefix + "shared.sg"].float().reshape(1, spec.width))
+        self.gates = len(rows) - 1                                    # the shared expert's gate: one more router row
         self.router = torch.cat(rows, dim=0).contiguous()             # float32: the router is computed in 32 bits
-        self.correction = tensors[prefix + "correction"].float().contiguous()
+        if p.get("router_bias", False) and (self.score != "picked" or p.get("correction", True)):
+            raise ValueError("routed feed-forward: a bias of the logits goes with the score 'picked' and no correction")
+        if p.get("correction", True):
+            self.correction = tensors[prefix + "correction"].float().contiguous()
+        elif p.get("router_bias", False):
+            self.correction = tensors[prefix + "router.b"].float().contiguous()
+        else:
+            self.correction = torch.zeros(n, dtype=torch.float32, device=self.router.device)
         self.w_up = self.w_down = None
         if E:
             if self.clamped:                   # [gate; up] rows of every expert
@@ -120,14 +149,25 @@ class RoutedFeedForward:
                 self.w_up = torch.stack([tensors[f"{prefix}e{e}.up"].to(ctx.dtype) for e in range(E)]).contiguous()
             self.w_down = torch.stack([tensors[f"{prefix}e{e}.down"].to(ctx.dtype) for e in range(E)]).contiguous()
 
-    def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
-        idx, wt, gate = K.moe_route(x, self.router, self.correction, self.E + self.I, 1 if self.shared else 0,
+    def _pieces(self, x: torch.Tensor, batch):
+        idx, wt, gate = K.moe_route(x, self.router, self.correction, self.E + self.I, self.gates,
                                     self.groups, self.keep, self.top, self.scale, self.score, self.group_score)
         y = None
         if self.E:
             y = self._experts(x, idx)
         s = self.shared.forward(x, batch) if self.shared is not None else None
+        return y, idx, wt, s, gate
+
+    def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
+        y, idx, wt, s, gate = self._pieces(x, batch)
         return K.moe_combine(y, idx, wt, x, s, gate, self.E)
+
+    def forward_pieces(self, x: torch.Tensor, batch):
+        """The output as the pieces of its weighted sum, for a caller whose next step takes them (see
+        ``RMSNorm.add_normed``); the output itself where there are identity experts or odd sizes."""
+        if self.I or not self.E or not K.moe_combine_norm_supported(x.shape[1]):
+            return self.forward(x, batch)
+        return PickedSum(*self._pieces(x, batch), n_experts=self.E)
 
     def _experts(self, x: torch.Tensor, idx: torch.Tensor) -> torch.Tensor:
         """float32 ``[pairs, width]``: every planned pair's expert output at the pair's own place."""

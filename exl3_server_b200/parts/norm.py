@@ -48,6 +48,7 @@ class RMSNorm:
         # a weight stored in 32-bit stays 32-bit; the kernel reads either
         self.weight = w.contiguous() if w.dtype == torch.float32 else w.to(ctx.dtype).contiguous()
         self.out_dtype = ctx.dtype
+        self._w32: Optional[torch.Tensor] = None
 
     offers_raw = True
 
@@ -68,12 +69,19 @@ class RMSNorm:
 
     def add_normed(self, stream: ResidualStream, y: Optional[torch.Tensor], want_x: bool = True) -> Optional[torch.Tensor]:
         """The norm on a sublayer's OUTPUT: ``h += y * rsqrt(mean(y^2) + eps) * w`` in float32; returns the new
-        residual in the activation type, which the next sublayer reads (``h`` itself in the float32 path).  With
+        residual in the activation type, which the next sublayer reads (``h`` itself in the float32 path).  ``y`` may
+        be a sum in pieces (``parts/moe.py``, ``PickedSum``).  With
         ``y`` None nothing is added and the residual is only handed over.  ``want_x`` False: nothing is returned
         (the next sublayer reads a norm of the residual, not the residual)."""
         if stream.pending is not None:
             raise RuntimeError("the residual stream holds an output that was not folded in")
         stream.normed = None
+        if hasattr(y, "norm_add"):
+            # a weighted sum in pieces: summed, normed and added in one kernel
+            bf16 = want_x and self.out_dtype == torch.bfloat16
+            x = y.norm_add(stream.h, self._weight32(), self.spec.eps, bf16)
+            stream.act = (x if bf16 else stream.h) if want_x else None
+            return stream.act
         if not want_x:
             stream.act = None
             K.norm_add(stream.h, y, self.weight, self.spec.eps, None)
@@ -92,6 +100,13 @@ class RMSNorm:
                             then_norm.out_dtype)
         stream.act = None
         stream.normed = (then_norm, ReadyNormed(x))
+
+    def _weight32(self) -> torch.Tensor:
+        if self.weight.dtype != torch.float32:
+            if self._w32 is None:
+                self._w32 = self.weight.float().contiguous()
+            return self._w32
+        return self.weight
 
     def fuse_args(self):
         """``(weight, eps, width)`` for a projection kernel that prepares this norm (see ``NormAfter``)."""

@@ -4,8 +4,11 @@ Per token ``q, k, v = r Wq^T, r Wk^T, r Wv^T`` (one joint matrix; biases optiona
 ``kv_heads`` key/value heads (query head h reads key/value head ``h // (heads / kv_heads)``), keys and queries of
 ``head_dim`` features, values of ``value_dim``.  Then, each an option of the spec's ``params``:
 
-* ``qk_norm``: ``"none"``, ``"unit"`` (each query and key head divided by its root mean square) or ``"weight"``
-  (the same times a weight ``[head_dim]`` shared by all heads), with ``norm_eps``, before the rotation;
+* ``qk_norm``: ``"none"``, ``"unit"`` (each query and key head divided by its root mean square), ``"weight"``
+  (the same times a weight ``[head_dim]`` shared by all heads) or ``"rows"`` (all query heads of a token divided by
+  their common root mean square, times a weight ``[heads * head_dim]``; the key heads likewise), with ``norm_eps``,
+  before the rotation;
+* ``q_temp``: ``(coef, every)``; queries at position p are multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``;
 * the position encoding of the spec (``rope`` with its layout, partial rotation and stretched table, or none);
 * ``v_mix``: ``"source"`` leaves this layer's values (before any mixing) for later layers of the same
   ``v_mix_key``; ``"mix"`` replaces ``v`` by ``(1 - lambda) v + lambda v_source`` with a learned scalar; the mixed
@@ -15,6 +18,11 @@ Per token ``q, k, v = r Wq^T, r Wk^T, r Wv^T`` (one joint matrix; biases optiona
 * ``window`` of the spec > 0: a query sees the last ``window`` keys, and with ``keep_first`` > 0 also the keys at
   positions below ``keep_first`` (at their true positions);
 * ``softcap`` > 0: the scaled scores become ``softcap * tanh(score / softcap)``;
+* ``distance_bias``: the largest distance of a learned table ``rel [rows, heads]`` of score biases by distance (see
+  ``parts/distance_bias.py``), added to the scores after scale and cap;
+* ``reads_kv``: the layer has no keys and values of its own; its schedule entry names the entry whose cache it reads;
+* ``tile_rows``: in bfloat16, key and value rows of up to 64 (128) features are kept 64 (128) wide in the cache, the rest
+  zeros, so that every such head size is the tensor-core kernels';
 * ``bias``: ``True`` (q, k, v and o have biases) or ``"qkv"`` (the output projection has none);
 * ``chunk`` > 0: a query sees only the causal keys of its own block of ``chunk`` positions (counted from the
   sequence's start, however the prompt was cut);
@@ -23,14 +31,14 @@ Per token ``q, k, v = r Wq^T, r Wk^T, r Wv^T`` (one joint matrix; biases optiona
 ``y = concat_h(o_h) Wo^T`` (+ bias).  Norms, rotation, mixing, scores and softmax are float32.  One kernel
 (``kernels.qk_prep``) does everything between the projection and the attention and writes the cache.  In bfloat16
 with keys and values of 64 or 128 features the attention is the tensor-core kernels' (tcgen05 for prompts, which
-takes every option above; the TMA page stream for steps of few tokens, which takes the sink of score 0 and the blocks
-but no window, cap or learned sink); everything else (float32,
+takes every option above; the TMA page stream for steps of few tokens, which takes sinks, distance biases and the blocks
+but no window and no cap); everything else (float32,
 other sizes, values of another width than keys) is the CUDA-core kernel in its general form
 (``kernels.attn_tokens_ex``), the same for prompts, portions of prompts and single tokens.  Head sizes are padded to
 a multiple of 8 in the cache (zeros), so any even size runs.
 
 Tensor names under the mixer's prefix: ``q``, ``k``, ``v``, ``o`` (biases: the name + ``.b``), ``q.norm``,
-``k.norm``, ``vmix``.
+``k.norm``, ``vmix``, ``sink``, ``rel``.
 
 A mixer of this kind can also run on a slice of a projection that another part computed together with other
 inputs' (``input_weight`` / ``forward_projected``; see ``parts/parallel.py``).
@@ -45,15 +53,21 @@ from ..ops import kernels as K
 from ..weights.loader import TensorSpec
 from .attention import BUSY_ITEMS, SPLIT_KEYS, Attention
 from .base import BuildContext, KVRequest, StateRequest
+from .distance_bias import DistanceBias
 from .linear import Linear
 from .registry import position_class, register_mixer
 from .spec import MixerSpec, PositionSpec
 
-NORM_CODES = {"none": 0, "unit": 1, "weight": 2}
+NORM_CODES = {"none": 0, "unit": 1, "weight": 2, "rows": 3}
 
 
 def pad8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+def tile_row(d: int, dv: int) -> int:
+    """The row width of the tensor-core kernels that holds keys of d and values of dv features; 0: too wide for them."""
+    return next((row for row in (64, 128) if max(d, dv) <= row), 0)
 
 
 class NormedAttention:
@@ -62,20 +76,29 @@ class NormedAttention:
         dv = int(spec.params.get("value_dim", 0)) or spec.head_dim
         return spec.heads, spec.kv_heads, spec.head_dim, dv
 
+    @staticmethod
+    def _projected(spec: MixerSpec) -> Tuple[str, ...]:
+        return ("q",) if spec.params.get("reads_kv", False) else ("q", "k", "v")
+
     @classmethod
     def tensor_specs(cls, spec: MixerSpec, prefix: str) -> List[TensorSpec]:
         H, G, d, dv = cls._sizes(spec)
-        out = [TensorSpec(prefix + "q", (H * d, spec.width)), TensorSpec(prefix + "k", (G * d, spec.width)),
-               TensorSpec(prefix + "v", (G * dv, spec.width)), TensorSpec(prefix + "o", (spec.width, H * dv))]
+        rows = {"q": H * d, "k": G * d, "v": G * dv}
+        names = cls._projected(spec)
+        out = [TensorSpec(prefix + n, (rows[n], spec.width)) for n in names]
+        out.append(TensorSpec(prefix + "o", (spec.width, H * dv)))
         if spec.params.get("bias", False):
-            out += [TensorSpec(prefix + "q.b", (H * d,)), TensorSpec(prefix + "k.b", (G * d,)),
-                    TensorSpec(prefix + "v.b", (G * dv,))]
+            out += [TensorSpec(prefix + n + ".b", (rows[n],)) for n in names]
             if spec.params["bias"] != "qkv":
                 out.append(TensorSpec(prefix + "o.b", (spec.width,)))
         if spec.params.get("sink") == "learned":
             out.append(TensorSpec(prefix + "sink", (H,)))
-        if spec.params.get("qk_norm", "none") == "weight":
-            out += [TensorSpec(prefix + "q.norm", (d,), init="ones"), TensorSpec(prefix + "k.norm", (d,), init="ones")]
+        kind = spec.params.get("qk_norm", "none")
+        if kind in ("weight", "rows"):
+            out += [TensorSpec(prefix + n + ".norm", (d if kind == "weight" else rows[n],), init="ones")
+                    for n in names if n != "v"]
+        if spec.params.get("distance_bias") is not None:
+            out.append(DistanceBias.tensor_spec(prefix + "rel", H))
         if spec.params.get("v_mix") in ("source", "mix"):
             out.append(TensorSpec(prefix + "vmix", ()))           # the source layer stores one too and never uses it
         return out
@@ -88,10 +111,23 @@ class NormedAttention:
         self.spec, self.ctx = spec, ctx
         self.H, self.G, self.d, self.dv = H, G, d, dv
         self.d_pad, self.dv_pad = pad8(d), pad8(dv)
+        if p.get("tile_rows", False) and ctx.dtype == torch.bfloat16 and tile_row(d, dv):
+            self.d_pad = self.dv_pad = tile_row(d, dv)
+        self.reads_kv = bool(p.get("reads_kv", False))
+        self.q_temp = tuple(float(x) for x in p["q_temp"]) if p.get("q_temp") else None
         self.norm = NORM_CODES[p.get("qk_norm", "none")]
         self.eps = float(p.get("norm_eps", 1e-6))
         self.sink = bool(p.get("sink", False))
         self.sink_vals = tensors[prefix + "sink"].float().contiguous() if p.get("sink") == "learned" else None
+        self.dist: Optional[torch.Tensor] = None
+        if p.get("distance_bias") is not None:
+            # the softmax does not see a constant added to every score: the table is kept relative to what the farthest
+            # keys get, so that only near keys carry a bias, and the sink's score moves along
+            bias = DistanceBias(tensors[prefix + "rel"], p["distance_bias"])
+            self.dist = K.distance_table(bias.near).to(ctx.device)
+            if self.sink:
+                base = self.sink_vals.double() if self.sink_vals is not None else torch.zeros_like(bias.far)
+                self.sink_vals = (base - bias.far.to(base.device)).float().to(ctx.device).contiguous()
         self.chunk = int(p.get("chunk", 0))
         self.window = int(spec.window)
         self.keep_first = int(p.get("keep_first", 0)) if self.window > 0 else 0
@@ -102,16 +138,17 @@ class NormedAttention:
         self.v_mix_key = ("v_mix", p.get("v_mix_key", 0))
         self.scale = spec.softmax_scale if spec.softmax_scale is not None else d ** -0.5
         bias = bool(p.get("bias", False))
-        self._w = torch.cat([tensors[prefix + n].to(ctx.dtype) for n in ("q", "k", "v")], dim=0)
-        self._b = torch.cat([tensors[prefix + n + ".b"].to(ctx.dtype) for n in ("q", "k", "v")]) if bias else None
+        names = self._projected(spec)
+        self._w = torch.cat([tensors[prefix + n].to(ctx.dtype) for n in names], dim=0)
+        self._b = torch.cat([tensors[prefix + n + ".b"].to(ctx.dtype) for n in names]) if bias else None
         self.n_proj = self._w.shape[0]
         self.qkv: Optional[Linear] = None                   # made on first use: a parallel part may project for us
         wo = tensors[prefix + "o"].to(ctx.dtype)
         if self.dv_pad != dv:                               # the attention's rows are padded: zero columns for the pad
             wo = torch.nn.functional.pad(wo.view(spec.width, H, dv), (0, self.dv_pad - dv)).reshape(spec.width, -1)
         self.o = Linear(wo, tensors[prefix + "o.b"] if bias and p["bias"] != "qkv" else None, ctx.dtype)
-        self.q_w = tensors[prefix + "q.norm"].float().contiguous() if self.norm == 2 else None
-        self.k_w = tensors[prefix + "k.norm"].float().contiguous() if self.norm == 2 else None
+        self.q_w = tensors[prefix + "q.norm"].float().contiguous() if self.norm >= 2 else None
+        self.k_w = tensors[prefix + "k.norm"].float().contiguous() if self.norm >= 2 and not self.reads_kv else None
         self.lam = tensors[prefix + "vmix"].float().reshape(1).contiguous() if self.v_mix == "mix" else None
         pos = spec.position or PositionSpec(kind="none", dims=0)
         self.position = position_class(pos.kind)(pos, d, ctx)
@@ -121,8 +158,8 @@ class NormedAttention:
         self._cuts = Attention.__new__(Attention)
         self._cuts.spec = MixerSpec(kind="attention", width=spec.width, heads=H, kv_heads=G, head_dim=self.d_pad,
                                     window=self.chunk or (self.window + self.keep_first if self.window else 0))
-        # what the tensor-core kernels do not apply
-        self._plain_scores = self.window == 0 and self.softcap == 0.0 and self.sink_vals is None
+        # what the decode kernel does not apply
+        self._plain_scores = self.window == 0 and self.softcap == 0.0
 
     # -- what a part that projects for several mixers at once needs -----------------------------------------------
     def input_weight(self) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
@@ -143,8 +180,8 @@ class NormedAttention:
 
     def forward_projected(self, proj: torch.Tensor, off: int, batch, kv, state) -> torch.Tensor:
         """``proj [T, *]`` holds this mixer's ``[q | k | v]`` from column ``off`` on."""
-        if kv is None or not kv.owns:
-            raise RuntimeError("normed attention needs a cache view of its own")
+        if kv is None or kv.owns == self.reads_kv:
+            raise RuntimeError("normed attention needs a cache view of its own, or another layer's when it reads one")
         H, G, d, dv = self.H, self.G, self.d, self.dv
         T = proj.shape[0]
         q_off, k_off, v_off = off, off + H * d, off + (H + G) * d
@@ -156,10 +193,12 @@ class NormedAttention:
             if src is None:
                 raise RuntimeError("normed attention: no earlier layer left its values to mix in")
             mix = (self.lam, src)
-        q, _ = K.qk_prep(proj, q_off, k_off, v_off, H, G, d, dv, self.d_pad, self.dv_pad, self.norm, self.q_w, self.k_w,
-                         self.eps, self.rot, self.position.layout_code, self.position.table if self.rot else None,
-                         self.position.mscale, 1.0, mix, batch.tok_pos, batch.tok_seq, kv.block_table, kv.page_size,
-                         self.ctx.dtype, kv.k, kv.v)
+        own = not self.reads_kv
+        q, _ = K.qk_prep(proj, q_off, k_off if own else 0, v_off if own else -1, H, G if own else 0, d, dv, self.d_pad,
+                         self.dv_pad, self.norm, self.q_w, self.k_w, self.eps, self.rot, self.position.layout_code,
+                         self.position.table if self.rot else None, self.position.mscale, 1.0, mix, batch.tok_pos,
+                         batch.tok_seq, kv.block_table, kv.page_size, self.ctx.dtype, kv.k if own else None,
+                         kv.v if own else None, temperature=self.q_temp)
         out = torch.empty((T, H * self.dv_pad), dtype=self.ctx.dtype, device=proj.device)
         if self._tensor_cores(q, out, batch, kv):
             return self.o(out, out_dtype=self.o.wide_dtype(T))
@@ -177,16 +216,17 @@ class NormedAttention:
             scratch = batch.workspace.floats(K.attn_tokens_scratch_bytes(T, H, self.dv_pad, n) // 4)
         K.attn_tokens_ex(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.tok_pos, batch.tok_seq, T, H, G,
                          self.d_pad, self.dv_pad, kv.page_size, self.window, self.chunk, self.sink, self.scale, split, n,
-                         scratch, keep_first=self.keep_first, softcap=self.softcap, sink_vals=self.sink_vals)
+                         scratch, keep_first=self.keep_first, softcap=self.softcap, sink_vals=self.sink_vals,
+                         dist=self.dist)
         return self.o(out, out_dtype=self.o.wide_dtype(T))
 
     def _tensor_cores(self, q: torch.Tensor, out: torch.Tensor, batch, kv) -> bool:
         """bfloat16 with keys and values of 64 or 128 features: prompts through the tcgen05 kernel, steps of few
         tokens through the kernel that streams pages by TMA, both with the sink and the blocks of positions as
         parameters.  False when the sizes are not theirs (the CUDA-core kernel then takes the step)."""
-        if self.ctx.dtype != torch.bfloat16 or self.d_pad != self.dv_pad or self.d_pad != self.d:
+        if self.ctx.dtype != torch.bfloat16 or self.d_pad != self.dv_pad:
             return False
-        H, G, d, T = self.H, self.G, self.d, q.shape[0]
+        H, G, d, T = self.H, self.G, self.d_pad, q.shape[0]
         if batch.max_new > 1 and batch.tiles and K.attn_prefill_tc_supported(torch.bfloat16, d, kv.page_size):
             tile_seq, tile_q0, n_tiles = batch.tiles[128]
             key = ("attn_prefill_variant", H, d, self.chunk, self.window, self.keep_first)
@@ -196,10 +236,10 @@ class NormedAttention:
             K.attn_prefill_tc(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.row_start, batch.row_pos0, tile_seq,
                               tile_q0, n_tiles, H, G, d, kv.page_size, self.window, self.scale, variant=variant,
                               chunk=self.chunk, sink=self.sink, keep_first=self.keep_first, softcap=self.softcap,
-                              sink_vals=self.sink_vals)
+                              sink_vals=self.sink_vals, dist=self.dist)
             return True
         if not self._plain_scores:
-            return False                 # single tokens with a window, a cap or sink scores: the CUDA-core kernel
+            return False                 # single tokens with a window or a cap: the CUDA-core kernel
         if not K.attn_decode_supported(torch.bfloat16, T, H, G, d, kv.page_size, kv.page_size, 1):
             return False
         split, head_split, in_block = self._cuts._decode_split(T, batch.max_kv_len, kv.page_size, q.device)
@@ -210,7 +250,7 @@ class NormedAttention:
             scratch = batch.workspace.floats(K.attn_tokens_scratch_bytes(T, H, d, n) // 4)
         K.attn_decode(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.tok_pos, batch.tok_seq, T, H, G, d,
                       kv.page_size, 0, self.scale, split, n, scratch, head_split=head_split, in_block=in_block,
-                      twins=twins, chunk=self.chunk, sink=self.sink)
+                      twins=twins, chunk=self.chunk, sink=self.sink, sink_vals=self.sink_vals, dist=self.dist)
         return True
 
     def _chunks(self, max_kv_len: int, split: int) -> int:
