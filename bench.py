@@ -31,6 +31,7 @@ blocks beside retention, wkv recurrences, dense GELU layers) and the Nibelix
 decoder (lightning recurrences, differential attention over a window, dense and
 routed feed-forwards) and the Potodra decoder (a residual of four streams, attention over a window that keeps the first
 keys, matrix memories with exponential gates, a gated delta rule beside causal attention, dense and routed
+feed-forwards) and the Tunavik decoder (causal attention with distance biases, a sink and shared keys and values, routed
 feed-forwards) beside the Llama-family decoder at equal width, depth, head count and feed-forward width,
 with random weights: one prompt of
 ``--prefill-tokens`` tokens and decode steps at ``--batch`` and ``--context``,
@@ -194,6 +195,20 @@ def potodra_config(z):
     kinds = [("attention", att, moe), ("mlstm", memory, dense), ("parallel", par, dense), ("mlstm", memory, moe)]
     layers = [PotodraLayer(kinds[i % 4][0], dict(kinds[i % 4][1]), dict(kinds[i % 4][2])) for i in range(z["layers"])]
     return PotodraConfig(vocab=z["vocab"], width=z["width"], streams=4, norm_eps=1e-6, embedding_scale=2.0, layers=layers)
+
+
+def tunavik_config(z):
+    """Tunavik at one of the size pairs: every layer has the other sides' attention heads (causal, a bias for keys less than
+    256 positions back, a sink, one norm over all heads) and a routed feed-forward like the Nibelix and Potodra sides': 16
+    experts, 2 picks a token, experts and the shared expert a quarter of the dense feed-forward's width.  Every fourth layer
+    reads the keys and values of the one before."""
+    from exl3_server_b200.config.tunavik import TunavikConfig, TunavikLayer
+    hd = z["head_dim"]
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": hd, "vdim": hd, "scale": hd ** -0.5, "bias_max": 256,
+           "q_temp": {"coef": 0.1, "every": 2048}, "kv_from": None}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 2}, "shared": {"ff": z["ff"] // 4}}
+    layers = [TunavikLayer("attention", dict(att, kv_from=i - 1 if i % 4 == 3 else None), dict(moe)) for i in range(z["layers"])]
+    return TunavikConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, logit_scale=1.5, logit_softcap=30.0, layers=layers)
 
 
 def design_configs(name: str):
@@ -421,8 +436,8 @@ class Rig:
 
 
 def designs(args) -> int:
-    """``--only designs``: prefill and decode throughput of the Rigitar, Nikodra, Nibelix and Potodra decoders beside the Llama-family
-    decoder of equal sizes; one JSON line."""
+    """``--only designs``: prefill and decode throughput of the Rigitar, Nikodra, Nibelix, Potodra and Tunavik decoders beside
+    the Llama-family decoder of equal sizes; one JSON line."""
     import torch
     torch.cuda.set_device(0)
     hbm_gbs, bf16_tf, peak_src = peaks()
@@ -435,7 +450,7 @@ def designs(args) -> int:
     for name in ([args.design_sizes] if args.design_sizes else sorted(DESIGN_SIZES)):
         rig_cfg, llama_cfg = design_configs(name)
         rec = {}
-        for arch, cfg in (("potodra", potodra_config(DESIGN_SIZES[name])), ("nibelix", nibelix_config(DESIGN_SIZES[name])),
+        for arch, cfg in (("tunavik", tunavik_config(DESIGN_SIZES[name])), ("potodra", potodra_config(DESIGN_SIZES[name])), ("nibelix", nibelix_config(DESIGN_SIZES[name])),
                           ("nikodra", nikodra_config(DESIGN_SIZES[name])),
                           ("rigitar", rig_cfg), ("llama", llama_cfg)):
             if args.design_arch not in ("both", arch):
@@ -478,7 +493,7 @@ def main() -> int:
                     help="run one part only (for profiling small cases); prints a short JSON line")
     ap.add_argument("--design-sizes", choices=sorted(DESIGN_SIZES), default=None,
                     help="with --only designs: one size pair instead of all")
-    ap.add_argument("--design-arch", choices=["both", "potodra", "nibelix", "nikodra", "rigitar", "llama"], default="both",
+    ap.add_argument("--design-arch", choices=["both", "tunavik", "potodra", "nibelix", "nikodra", "rigitar", "llama"], default="both",
                     help="with --only designs: one of the designs only (both: all of them)")
     ap.add_argument("--design-part", choices=["both", "prefill", "decode"], default="both",
                     help="with --only designs: one of the two measurements only")
