@@ -466,7 +466,7 @@ moe_gather_kernel(const __nv_bfloat16* x, int64_t ldx, int top, const int* order
 // The weighted sum and the norm on it with the residual's step, in one kernel (a block a token): v = sum_k weight[t, k]
 // y[t, k] + gate[t] shared[t], h[t] += v / sqrt(mean(v^2) + eps) * w, x[t] = h[t] in x's type.  A thread keeps its pieces
 // of four values in registers: rows of up to CN_THREADS * 4 * CN_VECS values, a multiple of 4.  No identity picks.
-constexpr int CN_THREADS = 256, CN_VECS = 8;
+constexpr int CN_THREADS = 256, CN_VECS = 8, CN_PICKS = 4;     // picks whose rows are asked for together
 
 __device__ inline void cn_load4(const float* p, float (&v)[4]) { load_vec_cg(p, v); }
 __device__ inline void cn_load4(const __nv_bfloat16* p, float (&v)[4]) {
@@ -475,33 +475,66 @@ __device__ inline void cn_load4(const __nv_bfloat16* p, float (&v)[4]) {
   v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
 }
 
-template <typename TS>
+template <typename TS, int VECS>
 __global__ void __launch_bounds__(CN_THREADS)
 moe_combine_norm_kernel(const float* y, const int* idx, const float* wt, const TS* shared, const float* gate, float* h,
                         const float* __restrict__ w, float eps, __nv_bfloat16* x, int H, int top, int n_experts) {
   __shared__ float red[32];
-  pdl_wait();
-  pdl_trigger();
   const int t = blockIdx.x;
   const int64_t base = (int64_t)t * H;
-  float v[CN_VECS][4];
-  float ss = 0.0f;
+  float wv[VECS][4];                               // the norm's weight does not depend on the kernel before
+#pragma unroll
+  for (int p = 0; p < VECS; ++p) {
+    const int c = (p * CN_THREADS + threadIdx.x) * 4;
+    if (c < H) load_vec(w + c, wv[p]);
+  }
+  pdl_wait();
+  pdl_trigger();
+  float v[VECS][4], hv[VECS][4];
   const float gt = gate ? __ldcg(gate + t) : 1.0f;
 #pragma unroll
-  for (int p = 0; p < CN_VECS; ++p) {
+  for (int p = 0; p < VECS; ++p) {
+    const int c = (p * CN_THREADS + threadIdx.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[p][e] = 0.0f;
+    if (c < H) load_vec_cg(h + base + c, hv[p]);
+  }
+  for (int k0 = 0; k0 < top; k0 += CN_PICKS) {
+    float wk[CN_PICKS];
+#pragma unroll
+    for (int k = 0; k < CN_PICKS; ++k) {
+      wk[k] = 0.0f;
+      if (k0 + k < top) {
+        const int ex = __ldcg(idx + (int64_t)t * top + k0 + k);
+        const float wr = __ldcg(wt + (int64_t)t * top + k0 + k);
+        if (ex >= 0 && ex < n_experts) wk[k] = wr;
+      }
+    }
+#pragma unroll
+    for (int p = 0; p < VECS; ++p) {
+      const int c = (p * CN_THREADS + threadIdx.x) * 4;
+      if (c < H) {
+        float a[CN_PICKS][4];
+        // every pair of a token is planned where there are no identity picks; a pick of no expert has weight zero and
+        // its row, which nobody wrote, is not read
+#pragma unroll
+        for (int k = 0; k < CN_PICKS; ++k) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[k][e] = 0.0f;
+          if (k0 + k < top && wk[k] != 0.0f) load_vec_cg(y + ((int64_t)t * top + k0 + k) * H + c, a[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < CN_PICKS; ++k)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[p][e] = fmaf(wk[k], a[k][e], v[p][e]);
+      }
+    }
+  }
+  float ss = 0.0f;
+#pragma unroll
+  for (int p = 0; p < VECS; ++p) {
     const int c = (p * CN_THREADS + threadIdx.x) * 4;
     if (c < H) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) v[p][e] = 0.0f;
-      for (int k = 0; k < top; ++k) {
-        const int ex = __ldcg(idx + (int64_t)t * top + k);
-        if (ex < 0 || ex >= n_experts) continue;
-        const float wk = __ldcg(wt + (int64_t)t * top + k);
-        float a[4];
-        load_vec_cg(y + ((int64_t)t * top + k) * H + c, a);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) v[p][e] = fmaf(wk, a[e], v[p][e]);
-      }
       if (shared) {
         float a[4];
         cn_load4(shared + base + c, a);
@@ -514,14 +547,12 @@ moe_combine_norm_kernel(const float* y, const int* idx, const float* wt, const T
   }
   const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)H + eps);
 #pragma unroll
-  for (int p = 0; p < CN_VECS; ++p) {
+  for (int p = 0; p < VECS; ++p) {
     const int c = (p * CN_THREADS + threadIdx.x) * 4;
     if (c < H) {
-      float a[4], wv[4];
-      load_vec_cg(h + base + c, a);
-      load_vec(w + c, wv);
+      float a[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) a[e] += v[p][e] * inv * wv[e];
+      for (int e = 0; e < 4; ++e) a[e] = hv[p][e] + v[p][e] * inv * wv[p][e];
       store_vec(h + base + c, a);
       if (x) {
         __nv_bfloat162 lo = __floats2bfloat162_rn(a[0], a[1]), hi = __floats2bfloat162_rn(a[2], a[3]);
@@ -754,13 +785,14 @@ extern "C" int exl3_moe_combine_norm(const float* y, const int* idx, const float
               CN_THREADS * 4 * CN_VECS);
     return ERR_BAD_ARGUMENT;
   }
-  if (shared_dtype == DT_F32)
-    launch_pdl(moe_combine_norm_kernel<float>, dim3(T), dim3(CN_THREADS), 0, stream, y, idx, wt, static_cast<const float*>(shared),
-               gate, h, w, eps, static_cast<__nv_bfloat16*>(x), H, top, n_experts);
-  else if (shared_dtype == DT_BF16)
-    launch_pdl(moe_combine_norm_kernel<__nv_bfloat16>, dim3(T), dim3(CN_THREADS), 0, stream, y, idx, wt,
-               static_cast<const __nv_bfloat16*>(shared), gate, h, w, eps, static_cast<__nv_bfloat16*>(x), H, top, n_experts);
-  else { set_error("moe_combine_norm: unsupported element type %d", shared_dtype); return ERR_UNSUPPORTED; }
+  if (shared_dtype != DT_F32 && shared_dtype != DT_BF16) { set_error("moe_combine_norm: unsupported element type %d", shared_dtype); return ERR_UNSUPPORTED; }
+#define EXL3_CN(TS, VECS)                                                                                              \
+  launch_pdl(moe_combine_norm_kernel<TS, VECS>, dim3(T), dim3(CN_THREADS), 0, stream, y, idx, wt,                      \
+             static_cast<const TS*>(shared), gate, h, w, eps, static_cast<__nv_bfloat16*>(x), H, top, n_experts)
+  const int need = ceil_div(H, CN_THREADS * 4);
+  if (shared_dtype == DT_F32) { if (need <= 2) EXL3_CN(float, 2); else if (need <= 4) EXL3_CN(float, 4); else EXL3_CN(float, CN_VECS); }
+  else { if (need <= 2) EXL3_CN(__nv_bfloat16, 2); else if (need <= 4) EXL3_CN(__nv_bfloat16, 4); else EXL3_CN(__nv_bfloat16, CN_VECS); }
+#undef EXL3_CN
   return launch_status("moe_combine_norm");
 }
 
