@@ -330,7 +330,7 @@ def test_the_temperature_steps_where_it_should(folders, tmp_path, dtype):
 
 
 @pytest.mark.parametrize("name", ["mixed", "wide"])
-def test_the_batch_and_the_cutting_change_nothing_in_float32(folders, name):
+def test_the_batch_and_the_pages_change_nothing_in_float32(folders, name):
     """The same tokens alone and as one of several in a batch of other lengths, on other pages and slots: the same bits."""
     from exl3_server_b200 import StepEntry
     folder = folders[name]
