@@ -104,6 +104,7 @@ int exl3_embed_hashed(const int* ids, const int* tok_pos, const int* tok_seq, co
 //   1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).  nkv 0: queries only (v_off < 0, no cache).  rot > 0: rotary encoding of the first rot features (layout 0: feature i with
 //   i + rot / 2; 1: feature 2i with 2i + 1), sines and cosines times mscale.  Keys are then multiplied by k_mul.
 //   mix_lambda != null: v <- (1 - lambda) v + lambda v_src[t] (v_src [T, v_src_ld], its own type).
+//   gate_out != null: gate_out[t, h] = sigmoid(x[t, g_off + h]), float32 [T, nh].
 //   Queries go to q_out [T, nh * hd_pad]; keys and values to the paged cache (k_pool / v_pool, rows of hd_pad /
 //   hdv_pad features, pad features zero), or, when k_pool is null, keys to k_out [T, nkv * hd_pad].
 int exl3_qk_prep(const void* x, int x_dtype, int64_t ld, int q_off, int k_off, int v_off, int T, int nh, int nkv,
@@ -112,7 +113,7 @@ int exl3_qk_prep(const void* x, int x_dtype, int64_t ld, int q_off, int k_off, i
                  float k_mul, const void* mix_lambda, int lambda_dtype, const void* v_src, int v_src_dtype,
                  int64_t v_src_ld, const int* tok_pos, const int* tok_seq, const int* block_table, int bt_stride,
                  int page, void* q_out, int q_out_dtype, void* k_out, int k_out_dtype, void* k_pool, void* v_pool,
-                 int pool_dtype, float temp_coef, float temp_every, cudaStream_t stream);
+                 int pool_dtype, float temp_coef, float temp_every, int g_off, float* gate_out, cudaStream_t stream);
 
 // Token shift: for s < n_mix, out[s][t] = h[t] + (h[t - 1] - h[t]) * mu[s]; the row before a row's first token of
 // this step comes from prev[slot] (float32 [slots, H], zero for a new sequence), which is then set to the row's last
@@ -189,22 +190,27 @@ int exl3_mingru_scan(const void* zug, int zug_dtype, void* y, int y_dtype, float
 //   cache row of token  = [ rmsnorm(a[:, kv_off : kv_off + kv_rank]) * wkv | 0 .. | rope(a[:, kv_off + kv_rank : + rot_dim]) | 0 .. ]
 //                         (the rotated part starts at rank_pad; the row is kv_row wide; skipped when pool is null)
 //   gate [T, heads]     = sigmoid(a[:, g_off : g_off + heads])  (float32)
-// The rotation takes the first rot features of the rot_dim part in half-split pairs at the token's position.
+//                         (heads 0 and gate null: none here)
+// The rotation takes the first rot features of the rot_dim part at the token's position: half-split pairs (layout 0) or
+// neighbours (1), sines and cosines times mscale.
 int exl3_latent_prep(const void* a, int a_dtype, int lda, int T, int q_off, int q_rank, const void* wq, int wq_dtype,
                      int kv_off, int kv_rank, int rot_dim, const void* wkv, int wkv_dtype, int g_off, int heads, float eps,
-                     const float* inv_freq, const float* inv_freq_lo, int rot, const int* tok_pos, const int* tok_seq,
-                     const int* block_table, int bt_stride, int page, void* pool, int pool_dtype, int kv_row,
+                     const float* inv_freq, const float* inv_freq_lo, int rot, int layout, float mscale, const int* tok_pos,
+                     const int* tok_seq, const int* block_table, int bt_stride, int page, void* pool, int pool_dtype, int kv_row,
                      int rank_pad, void* cq, int cq_dtype, float* gate, cudaStream_t stream);
 // Products per head: out[t, h, n] = mul[t, h] * sum_k x[t, h, k] * w[h, k, n]  (n < N, k < K; mul null: 1), with
 // x[t, h, k] at x + t * x_row + h * x_head + k and out likewise; float32 sums in the order of k.  With rot_dim > 0 the
 // rot_dim features of x that follow a head's K are rotated (first rot of them, half-split pairs, at the token's
 // position) and written behind the head's outputs at out[t, h, tail_off ..]; what lies between N and tail_off and
 // behind the tail up to out_head is set to zero.  x, w and out have one element type.  With w null only the tails are
-// written (the products come from elsewhere).
+// written (the products come from elsewhere).  gate (or null): logits [T, gate_row] whose sigmoid at h * N + n is one more
+// factor of out[t, h, n].  exl3_sigmoid_mul: y[t, i] *= sigmoid(g[t, i]).
 int exl3_head_gemm(const void* x, int64_t x_row, int x_head, const void* w, void* out, int64_t out_row, int out_head,
-                   int dtype, int T, int heads, int K, int N, const float* mul, int rot_dim, int rot,
-                   const float* inv_freq, const float* inv_freq_lo, const int* tok_pos, int tail_off,
+                   int dtype, int T, int heads, int K, int N, const float* mul, const void* gate, int gate_dtype,
+                   int64_t gate_row, int rot_dim, int rot, int layout, float mscale, const float* inv_freq, const float* inv_freq_lo, const int* tok_pos, int tail_off,
                    cudaStream_t stream);
+
+int exl3_sigmoid_mul(void* y, int dtype, const void* g, int g_dtype, int64_t g_row, int T, int n, cudaStream_t stream);
 
 size_t exl3_argmax_scratch_bytes(int R, int V);
 // Whole prompts on tcgen05 tensor cores with TMA loads from the paged cache (bfloat16, heads of 64 or 128, pages
@@ -277,7 +283,8 @@ int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, void* k_poo
                      const int* tok_seq, int T, int nh, int nkv, int hd, int page, int window, int chunk, int sink,
                      float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes, const float* inv_freq,
                      const float* inv_freq_lo, int rot, float pos_scale, int write_new, int head_split, int in_block,
-                     int twins, const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream);
+                     int twins, const float* sink_vals, const float* dist, int dist_len, const float* gate,
+                     cudaStream_t stream);
 
 int exl3_argmax(const float* logits, int* out, int R, int V, void* scratch, size_t scratch_bytes,
                 cudaStream_t stream);
@@ -303,7 +310,8 @@ int exl3_tanh_norm_add(float* h, const void* a, int a_dtype, const void* b, int 
 // A routed feed-forward (see moe.cu).  exl3_moe_route: wr float32 [E + extra, W]; idx int32 and wt float32 [T, top];
 // gate_out float32 [T] = sigmoid of the extra row.  exl3_moe_plan: order int32 [P], plan int32 [4 + 3 * max tiles].
 // exl3_moe_gemm: out[p] = act(W[e(p)] A[p / a_div]) for the planned pairs, W [n_experts, N, K]; act 0 none, 1 gelu
-// (exact), 2 gelu by the tanh formula, 3 silu, 4 the square of relu.  score_kind: 0 softmax, 1 sigmoid, + 2 groups scored
+// (exact), 2 gelu by the tanh formula, 3 silu, 4 the square of relu; + 16: rows of W alternate between a gate's and an up
+// projection's, out[p] is [N / 2] wide, act(gate) * up (also in exl3_moe_gemv and exl3_moe_gemm_tc).  score_kind: 0 softmax, 1 sigmoid, + 2 groups scored
 // by their two largest, 4 the softmax over the picks alone (corr is then a bias of the logits).  exl3_moe_combine: the weighted sum, float32 [T, H]; picks from
 // n_experts on stand for the input x itself; shared (any type) is added times gate (null: as it is).
 // exl3_moe_gemv: the same product for plans of tiles of at most exl3_moe_gemv_rows() rows (decode), bfloat16 A and W.
@@ -326,6 +334,10 @@ int exl3_moe_route(const void* x, int x_dtype, int64_t ldx, const float* wr, con
                    int extra, int groups, int keep, int top, float scale, int score_kind, int* idx, float* wt,
                    float* gate_out, cudaStream_t stream);
 int exl3_moe_plan(const int* idx, int P, int n_experts, int tile_rows, int* order, int* plan, cudaStream_t stream);
+// The plans of several layers whose experts come from tables by token id, in one launch: layer l's pair p = t * top[l] + k
+// goes to expert tables[l][ids[t] * top[l] + k] (host arrays of n_layers entries).
+int exl3_moe_table_plans(const int* ids, int T, int n_layers, const int* const* tables, const int* top, const int* n_experts,
+                         const int* tile_rows, int* const* order, int* const* plan, cudaStream_t stream);
 int exl3_moe_gemm(const void* A, int a_dtype, int64_t lda, int a_div, const void* W, int w_dtype, const int* order,
                   const int* plan, void* out, int out_dtype, int P, int n_experts, int N, int K, int act,
                   cudaStream_t stream);
@@ -352,13 +364,14 @@ int exl3_diff_combine(const void* a, int a_dtype, int a_row, const void* gate, i
 // replaces a score s (after the scale) by softcap * tanh(s / softcap); sink_vals [heads] (float32, with sink) are the
 // sink's scores per query head instead of 0; dist (dist_len > 0): biases per query head and distance, added to the scores
 // (after scale and cap) of keys less than dist_len positions back, a row per head of dist_len + 2 * DIST_PAD floats
-// (common.cuh).  max_splits must count the chunks of the kept keys too.
+// (common.cuh); gate: a factor per (token, query head) on the output, float32 [T, nh] (the tensor-core kernels take it
+// too).  max_splits must count the chunks of the kept keys too.
 int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* out, int out_f32, int dtype, const void* k_pool,
                          const void* v_pool, const int* block_table, int bt_stride, const int* tok_pos,
                          const int* tok_seq, int T, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                          int window, int chunk, int sink, float scale, int split_keys, int max_splits, float* scratch,
                          size_t scratch_bytes, int keep_first, float softcap, const float* sink_vals, const float* dist,
-                         int dist_len, cudaStream_t stream);
+                         int dist_len, const float* gate, cudaStream_t stream);
 
 // rows of gu are [gate (I) | up (I)], ld elements apart: out = g * sigmoid(alpha g) * (u + 1) with g = min(gate, limit)
 // and u = clamp(up, -limit, limit).
@@ -398,11 +411,17 @@ int exl3_conv_prep(const void* x, int x_dtype, int64_t ldx, int q_off, int k_off
 // out = sa * a + sb * b element by element, float32 out.
 int exl3_scaled_sum2(const void* a, const void* b, int ab_dtype, float sa, float sb, float* out, int64_t n,
                      cudaStream_t stream);
+// The residual's step between two layers (see residual_step.cu): h += scale * (a + b + pick_weight * sum_k picks[t, k]) +
+// emb_scale * emb[ids[t]] + vec, and, with w given, x = rmsnorm(h) * w.  Null pieces are skipped; ids null: row t of emb.
+int exl3_residual_step(float* h, const void* a, int a_dtype, const void* b, int b_dtype, const float* picks, int top,
+                       float pick_weight, float scale, const void* emb, int emb_dtype, const int* ids, float emb_scale,
+                       const float* vec, const void* w, int w_dtype, float eps, void* x, int x_dtype, int T, int H,
+                       cudaStream_t stream);
 int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int T, void* out, const void* k_pool, const void* v_pool,
                              int64_t n_pool_rows, const int* block_table, int bt_stride, const int* row_start,
                              const int* row_pos0, const int* tile_seq, const int* tile_q0, int n_tiles, int nh, int nkv,
                              int hd, int page, int window, int chunk, int sink, float scale, int variant, int keep_first,
-                             float softcap, const float* sink_vals, const float* dist, int dist_len,
+                             float softcap, const float* sink_vals, const float* dist, int dist_len, const float* gate,
                              cudaStream_t stream);
 // h[t] = table[ids[t]] * scale + a sinusoid of position tok_pos[t] (entry 2i: sin(p f_i), 2i + 1: cos(p f_i), f given as
 // float32 and what float32 lost, ceil(H / 2) each), then, with norm_w (float32 [H]) given, h / sqrt(mean(h^2) + eps) *

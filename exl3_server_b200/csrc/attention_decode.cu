@@ -190,6 +190,7 @@ struct AdOpts {
   const float* dist;                                     // biases per query head and distance; dist_len 0: none
   int dist_len;
   float dist_mul;                                        // 1 / scale: the biases join the scores before the scale
+  const float* gate;                                     // a factor per (token, query head) on the output; null: none
 };
 
 template <int HD, int NC, int TW>
@@ -287,6 +288,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
   auto sink_term = [&](int head, float m) {
     return ad_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m);
   };
+  auto out_factor = [&](int t, int head) { return opts.gate ? __ldcg(opts.gate + (int64_t)t * nh + head) : 1.0f; };
   auto chunks_of = [&](int t) { return s_cum[t + 1] - s_cum[t]; };
   auto base_of = [&](int t, int g) { return nkv * s_cum[t] + g * chunks_of(t); };   // index of chunk 0 of (t, g)
   // This warp's share: chunks i0 .. i1 - 1 of the list ordered by token, kv head, chunk: an equal contiguous share
@@ -537,7 +539,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         }
         ll = warp_sum(ll);
         if (sink) ll += sink_term(mg * G + n0 + n, M);
-        if (nn == n) my_ll = ll;
+        if (nn == n) my_ll = ll / out_factor(mt, mg * G + n0 + n);
       }
     }
     __syncwarp();
@@ -829,7 +831,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
         if (n_rec == 1) {
           __nv_bfloat16* dst = out + ((int64_t)t * nh + head) * HD;
           // a sink is one more key without a value: a term in the sum
-          const float inv = 1.0f / (sink ? l[c][h] + sink_term(head, m[c][h]) : l[c][h]);
+          const float inv = out_factor(t, head) / (sink ? l[c][h] + sink_term(head, m[c][h]) : l[c][h]);
 #pragma unroll
           for (int d = 0; d < NJ; ++d) {
             dst[16 * d + gl] = __float2bfloat16(o[c][d][h] * inv);
@@ -894,6 +896,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
           ll += s2 < n_rec ? rec_at(hb, s2, HD + 1) * w[s2] : 0.0f;
         }
         if (sink) ll += sink_term(g_blk * G + n, M);
+        ll /= out_factor(t_blk, g_blk * G + n);
         __nv_bfloat16* dst = out + ((int64_t)t_blk * nh + g_blk * G + n) * HD;
 #pragma unroll
         for (int e = 0; e < HD / 32; ++e) {
@@ -1003,7 +1006,7 @@ extern "C" int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, 
                                 float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes,
                                 const float* inv_freq, const float* inv_freq_lo, int rot, float pos_scale,
                                 int write_new, int head_split, int in_block, int twins, const float* sink_vals,
-                                const float* dist, int dist_len, cudaStream_t stream) {
+                                const float* dist, int dist_len, const float* gate, cudaStream_t stream) {
   if (T == 0) return 0;
   if (dist_len < 0 || (dist_len > 0 && dist == nullptr) || (sink_vals != nullptr && !sink)) {
     set_error("attn_decode: a table of %d distance biases is missing, or sink scores come without the sink", dist_len);
@@ -1069,6 +1072,7 @@ extern "C" int exl3_attn_decode(const void* q, int64_t q_row_stride, void* out, 
   opts.dist = dist;
   opts.dist_len = dist_len;
   opts.dist_mul = 1.0f / scale;
+  opts.gate = gate;
   // a stage is a page (heads of 64) or half a page (heads of 128): the copy's box has as many rows
   const int box_rows = hd == 64 ? 64 : 32;
   CUtensorMap map_k, map_v;

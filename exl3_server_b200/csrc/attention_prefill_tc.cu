@@ -185,6 +185,7 @@ struct FaOpts {
   const float* dist;
   int dist_len;
   float dist_mul;
+  const float* gate;           // a factor per (token, query head) on the output; null: none
 };
 // Whether a page of keys from key0 on holds a key with a bias for one of a warp's 32 queries from position p0 on.
 __device__ inline bool fa_near(int key0, int p0, int dist_len) {
@@ -537,7 +538,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       if (ok) {
         fa_fence_after();
         // a sink is a key of score 0 without a value: one more term in the sum, in the units of the reference maximum
-        const float inv = 1.0f / (sink ? l_run + fa_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m_used) : l_run);
+        float inv = 1.0f / (sink ? l_run + fa_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m_used) : l_run);
+        if (opts.gate && r < rows) inv *= __ldcg(opts.gate + (int64_t)(tw.row0 + r) * nh + head);
         __nv_bfloat16* dst = out + ((int64_t)(tw.row0 + r) * nh + head) * FA_HD;
 #pragma unroll
         for (int h2 = 0; h2 < FA_HD / 64; ++h2) {            // 64 columns at a time (every thread reads: the load is the warp's)
@@ -792,7 +794,8 @@ attn_prefill_tc4_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       ok = fa_mbar_wait(pv_done, jl & 1);
       if (ok) {
         fa_fence_after();
-        const float inv = 1.0f / (sink ? l_run + fa_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m_used) : l_run);
+        float inv = 1.0f / (sink ? l_run + fa_exp2((opts.sink_vals ? __ldg(opts.sink_vals + head) * 1.4426950408889634f : 0.0f) - m_used) : l_run);
+        if (opts.gate && r < rows) inv *= __ldcg(opts.gate + (int64_t)(row_start[b] + q0 + r) * nh + head);
         __nv_bfloat16* dst = out + ((int64_t)(row_start[b] + q0 + r) * nh + head) * 64;
 #pragma unroll 1
         for (int c0 = 0; c0 < 64; c0 += 32) {
@@ -879,7 +882,8 @@ extern "C" int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int
                                         const int* row_start, const int* row_pos0, const int* tile_seq,
                                         const int* tile_q0, int n_tiles, int nh, int nkv, int hd, int page, int window,
                                         int chunk, int sink, float scale, int variant, int keep_first, float softcap,
-                                        const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream) {
+                                        const float* sink_vals, const float* dist, int dist_len, const float* gate,
+                                        cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   if (dist_len < 0 || (dist_len > 0 && dist == nullptr)) {
     set_error("attn_prefill_tc: a table of %d distance biases is missing", dist_len);
@@ -897,6 +901,7 @@ extern "C" int exl3_attn_prefill_tc_opt(const void* q, int64_t q_row_stride, int
   opts.sink_vals = sink_vals;
   opts.dist = dist;
   opts.dist_len = dist_len;
+  opts.gate = gate;
   opts.dist_mul = softcap > 0.0f ? 1.0f / softcap : 1.0f / scale;
   if (!exl3_attn_prefill_tc_supported(DT_BF16, hd, page)) {
     set_error("attn_prefill_tc: needs bfloat16, head_dim 64 or 128 and pages of 64, got head_dim %d page %d", hd, page);
@@ -964,5 +969,5 @@ extern "C" int exl3_attn_prefill_tc(const void* q, int64_t q_row_stride, int T, 
                                     int chunk, int sink, float scale, int variant, cudaStream_t stream) {
   return exl3_attn_prefill_tc_opt(q, q_row_stride, T, out, k_pool, v_pool, n_pool_rows, block_table, bt_stride, row_start,
                                   row_pos0, tile_seq, tile_q0, n_tiles, nh, nkv, hd, page, window, chunk, sink, scale,
-                                  variant, 0, 0.0f, nullptr, nullptr, 0, stream);
+                                  variant, 0, 0.0f, nullptr, nullptr, 0, nullptr, stream);
 }

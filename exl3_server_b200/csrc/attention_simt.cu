@@ -30,12 +30,13 @@
 //              counted from the start of the sequence), on top of the causal bound and the window;
 //   sink:      one is added to the softmax's denominator, as if there were one more key with score 0 and a value
 //              of zero: p_j = exp(s_j) / (1 + sum_j exp(s_j)).
-// The entry point with every option (exl3_attn_tokens_opt) takes four more:
+// The entry point with every option (exl3_attn_tokens_opt) takes five more:
 //   keep_first > 0: with a window, the keys at positions below keep_first stay visible to every later query (at their
 //              true positions): j is seen when j <= pos and (pos - j < window or j < keep_first);
 //   softcap > 0: s <- softcap * tanh(s / softcap) after the scale;
 //   sink_vals: with sink, the sink's score per query head (not scaled, not capped) instead of 0:
 //              p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j));
+//   gate:      a float32 factor per (token, query head), [T, heads], on the output;
 //   dist:      s <- s + dist_h[pos - j] after the scale and the cap, for keys up to dist_len - 1 positions back (a
 //              table per query head; nothing is added further back).  Its layout is common.cuh's DIST_PAD.
 #include "api.h"
@@ -110,7 +111,8 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
                    const int* __restrict__ tok_seq, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                    int window, int chunk, int sink, float scale, int split_keys, int max_splits,
                    float* __restrict__ scratch, int* __restrict__ counters, int lpk, int out_f32, int keep_first,
-                   float softcap, const float* __restrict__ sink_vals, const float* __restrict__ dist, int dist_len) {
+                   float softcap, const float* __restrict__ sink_vals, const float* __restrict__ dist, int dist_len,
+                   const float* gate) {
   constexpr int VEC = Elem<T>::vec;
   constexpr int NA = R * VEC;
   constexpr int U = R == 1 ? 4 : (R == 2 ? 2 : 1);  // key groups whose loads are issued together
@@ -296,6 +298,7 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
       const int head = g * G + h0 + hh;
       if (max_splits <= 1) {
         if (sink) aa *= sink_finish<T>(mm, ll, sink_score<T>(sink_vals, head));
+        if (gate) aa *= __ldcg(gate + (int64_t)t * nh + head);
         att_store<T>(out, out_f32, ((int64_t)t * nh + head) * hdv + d, aa / ll);
       } else {
         float* sc = scratch + (((int64_t)t * nh + head) * max_splits + sp) * rec;
@@ -332,7 +335,8 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
     __syncthreads();
     float ll = 0.0f;
     for (int s2 = 0; s2 < max_splits; ++s2) ll += sl[s2] * sw[s2];
-    const float fin = sink ? sink_finish<T>(mx, ll, sink_score<T>(sink_vals, head)) : 1.0f;
+    float fin = sink ? sink_finish<T>(mx, ll, sink_score<T>(sink_vals, head)) : 1.0f;
+    if (gate) fin *= __ldcg(gate + (int64_t)t * nh + head);
     for (int d = threadIdx.x; d < hdv; d += blockDim.x) {
       float aa = 0.0f;
 #pragma unroll 4
@@ -348,7 +352,8 @@ attn_tokens_kernel(const T* __restrict__ q, int64_t q_row_stride, T* __restrict_
 // both sums in chunk order.  The records are read with independent loads.
 template <typename T>
 __global__ void attn_combine_kernel(const float* __restrict__ scratch, T* __restrict__ out, int nh, int hd,
-                                    int max_splits, int sink, int out_f32, const float* __restrict__ sink_vals) {
+                                    int max_splits, int sink, int out_f32, const float* __restrict__ sink_vals,
+                                    const float* gate) {
   extern __shared__ float sw[];                      // [max_splits] weights, then [max_splits] sums
   pdl_wait();
   pdl_trigger();
@@ -368,7 +373,8 @@ __global__ void attn_combine_kernel(const float* __restrict__ scratch, T* __rest
   __syncthreads();
   float ll = 0.0f;
   for (int s = 0; s < max_splits; ++s) ll += sl[s] * sw[s];
-  const float fin = sink ? sink_finish<T>(mx, ll, sink_score<T>(sink_vals, head)) : 1.0f;
+  float fin = sink ? sink_finish<T>(mx, ll, sink_score<T>(sink_vals, head)) : 1.0f;
+  if (gate) fin *= __ldcg(gate + (int64_t)t * nh + head);
   for (int d = threadIdx.x; d < hd; d += blockDim.x) {
     float aa = 0.0f;
 #pragma unroll 4
@@ -383,7 +389,7 @@ static int launch_tokens(const void* q, int64_t q_row_stride, void* out, const v
                          const int* tok_seq, int T_, int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page,
                          int window, int chunk, int sink, float scale, int split_keys, int max_splits, float* scratch, int lpk,
                          int out_f32, int keep_first, float softcap, const float* sink_vals, const float* dist, int dist_len,
-                         cudaStream_t stream) {
+                         const float* gate, cudaStream_t stream) {
   const size_t smem = ((size_t)ATT_WARPS * GT * (hdv + 2) + 2 * (size_t)max_splits) * sizeof(float);
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(attn_tokens_kernel<T, GT, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -403,12 +409,12 @@ static int launch_tokens(const void* q, int64_t q_row_stride, void* out, const v
              static_cast<const T*>(q), q_row_stride, static_cast<T*>(out), static_cast<const T*>(k_pool),
              static_cast<const T*>(v_pool), block_table, bt_stride, tok_pos, tok_seq, nh, nkv, hd, hdv, kv_row, v_row, page,
              window, chunk, sink, scale, split_keys, max_splits, scratch, counters, lpk, out_f32, keep_first, softcap,
-             sink_vals, dist, dist_len);
+             sink_vals, dist, dist_len, gate);
   int rc = launch_status("attn_tokens");
   if (rc) return rc;
   if (max_splits > 1 && !fused_merge) {
     launch_pdl(attn_combine_kernel<T>, dim3(T_, nh), dim3(64), (size_t)2 * max_splits * sizeof(float), stream,
-               (const float*)scratch, static_cast<T*>(out), nh, hdv, max_splits, sink, out_f32, sink_vals);
+               (const float*)scratch, static_cast<T*>(out), nh, hdv, max_splits, sink, out_f32, sink_vals, gate);
     rc = launch_status("attn_combine");
   }
   return rc;
@@ -419,7 +425,7 @@ static int dispatch(const void* q, int64_t q_row_stride, void* out, const void* 
                     const int* block_table, int bt_stride, const int* tok_pos, const int* tok_seq, int T_,
                     int nh, int nkv, int hd, int hdv, int kv_row, int v_row, int page, int window, int chunk, int sink,
                     float scale, int split_keys, int max_splits, float* scratch, int out_f32, int keep_first, float softcap,
-                    const float* sink_vals, const float* dist, int dist_len, cudaStream_t stream) {
+                    const float* sink_vals, const float* dist, int dist_len, const float* gate, cudaStream_t stream) {
   constexpr int VEC = Elem<T>::vec;
   const int vecs = ceil_div(max(hd, hdv), VEC);       // 16-byte pieces of the wider of a key row and a value row
   int lpk = 1;
@@ -430,7 +436,7 @@ static int dispatch(const void* q, int64_t q_row_stride, void* out, const void* 
   return launch_tokens<T, GT, RR>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos, \
                                   tok_seq, T_, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, \
                                   split_keys, max_splits, scratch, lpk, out_f32, keep_first, softcap, sink_vals, \
-                                  dist, dist_len, stream)
+                                  dist, dist_len, gate, stream)
   if (R == 1) {
     if (G == 1) EXL3_ATT(1, 1);
     if (G == 2) EXL3_ATT(2, 1);
@@ -471,7 +477,7 @@ extern "C" int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* o
                                     int hd, int hdv, int kv_row, int v_row, int page, int window, int chunk, int sink,
                                     float scale, int split_keys, int max_splits, float* scratch, size_t scratch_bytes,
                                     int keep_first, float softcap, const float* sink_vals, const float* dist, int dist_len,
-                                    cudaStream_t stream) {
+                                    const float* gate, cudaStream_t stream) {
   if (T == 0) return 0;
   if (dist_len < 0 || (dist_len > 0 && dist == nullptr)) {
     set_error("attn_tokens: a table of %d distance biases is missing", dist_len);
@@ -508,12 +514,12 @@ extern "C" int exl3_attn_tokens_opt(const void* q, int64_t q_row_stride, void* o
   if (dtype == DT_F32)
     return dispatch<float>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos, tok_seq, T,
                            nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, split_keys, max_splits,
-                           scratch, out_f32, keep_first, softcap, sink_vals, dist, dist_len, stream);
+                           scratch, out_f32, keep_first, softcap, sink_vals, dist, dist_len, gate, stream);
   if (dtype == DT_BF16)
     return dispatch<__nv_bfloat16>(q, q_row_stride, out, k_pool, v_pool, block_table, bt_stride, tok_pos,
                                    tok_seq, T, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale,
                                    split_keys, max_splits, scratch, out_f32, keep_first, softcap, sink_vals,
-                                   dist, dist_len, stream);
+                                   dist, dist_len, gate, stream);
   set_error("attn_tokens: unsupported element type %d", dtype);
   return ERR_UNSUPPORTED;
 }
@@ -526,7 +532,7 @@ extern "C" int exl3_attn_tokens_wide(const void* q, int64_t q_row_stride, void* 
                                      cudaStream_t stream) {
   return exl3_attn_tokens_opt(q, q_row_stride, out, out_f32, dtype, k_pool, v_pool, block_table, bt_stride, tok_pos, tok_seq,
                               T, nh, nkv, hd, hdv, kv_row, v_row, page, window, chunk, sink, scale, split_keys, max_splits,
-                              scratch, scratch_bytes, 0, 0.0f, nullptr, nullptr, 0, stream);
+                              scratch, scratch_bytes, 0, 0.0f, nullptr, nullptr, 0, nullptr, stream);
 }
 
 extern "C" int exl3_attn_tokens_ex(const void* q, int64_t q_row_stride, void* out, int dtype,

@@ -8,10 +8,13 @@
 //            logits, the choice is made by z + bias and the weights are the softmax over the chosen logits alone, times
 //            scale.  One more row of Wr may follow the router's: its sigmoid is a
 //            gate per token (for a shared expert) that the same kernel leaves beside the picks.
+//            Instead of a router, a table of experts by token id (moe_table_plans): no scores, equal weights; the plans of
+//            all such layers of a step are one launch, since they depend on the token ids alone.
 //   plan     the pairs (token, pick) whose pick is an expert with weights, ordered by expert and cut into tiles of
 //            at most a given number of rows of one expert; everything stays on the device (no count reaches the host), so the
 //            step can be part of a recorded graph.
 //   experts  mid[p] = act(W_up[e] x[token(p)]),  y[p] = W_down[e] mid[p], a block per (tile, 64 output features);
+//            (act with the GLU bit: rows of W_up alternate between a gate's and an up projection's, mid = act(gate) * up);
 //            a row's sum walks K in order with one float32 accumulator, so it does not depend on the row's tile mates.
 //   sum      out[t] = sum_k weight[t, k] * (y[t, k], or x[t] itself when pick k is an identity output: those are the
 //            router outputs from n_experts on, which have no weights) + gate[t] * shared[t].
@@ -260,18 +263,15 @@ moe_route_few_kernel(const TX* x, int64_t ldx, const float* __restrict__ wr, con
 
 // One block.  plan[0]: number of tiles; plan[1]: planned pairs (places of `order` in use); then per tile (expert,
 // first place in `order`, rows), from plan[4] on.  Tiles hold at most tile_rows rows.
-__global__ void __launch_bounds__(1024)
-moe_plan_kernel(const int* idx, int P, int n_experts, int tile_rows, int* order, int* plan) {
-  extern __shared__ int ps[];                      // counts, offsets, cursors
-  int* counts = ps;
+template <typename ExpertOf>
+__device__ inline void moe_make_plan(ExpertOf expert_of, int P, int n_experts, int tile_rows, int* order, int* plan, int* ps) {
+  int* counts = ps;                                // counts, offsets, cursors
   int* offs = ps + n_experts;
   int* cursor = offs + n_experts;
-  pdl_wait();
-  pdl_trigger();
   for (int e = threadIdx.x; e < n_experts; e += blockDim.x) { counts[e] = 0; cursor[e] = 0; }
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
-    const int e = __ldcg(idx + p);
+    const int e = expert_of(p);
     if (e >= 0 && e < n_experts) atomicAdd(&counts[e], 1);
   }
   __syncthreads();
@@ -292,10 +292,39 @@ moe_plan_kernel(const int* idx, int P, int n_experts, int tile_rows, int* order,
   }
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
-    const int e = __ldcg(idx + p);
+    const int e = expert_of(p);
     if (e >= 0 && e < n_experts) order[offs[e] + atomicAdd(&cursor[e], 1)] = p;
   }
 }
+
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(const int* idx, int P, int n_experts, int tile_rows, int* order, int* plan) {
+  extern __shared__ int ps[];
+  pdl_wait();
+  pdl_trigger();
+  moe_make_plan([&](int p) { return __ldcg(idx + p); }, P, n_experts, tile_rows, order, plan, ps);
+}
+
+// Block l makes layer l's plan from its table.
+constexpr int MOE_TABLES = 48;                     // layers a launch takes
+struct MoeTables {
+  const int* table[MOE_TABLES];
+  int* order[MOE_TABLES];
+  int* plan[MOE_TABLES];
+  int top[MOE_TABLES], n_experts[MOE_TABLES], tile_rows[MOE_TABLES];
+};
+__global__ void __launch_bounds__(1024)
+moe_table_plans_kernel(const int* ids, int T, const __grid_constant__ MoeTables m) {
+  extern __shared__ int ps[];
+  pdl_wait();
+  pdl_trigger();
+  const int l = blockIdx.x, top = m.top[l];
+  const int* table = m.table[l];
+  moe_make_plan([&](int p) { return __ldg(table + (int64_t)__ldcg(ids + p / top) * top + p % top); }, T * top, m.n_experts[l],
+                m.tile_rows[l], m.order[l], m.plan[l], ps);
+}
+
+constexpr int MOE_GLU = 16;                         // bit of act: act(even output) * (the odd output after it)
 
 __device__ inline float moe_act(float v, int act) {
   if (act == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
@@ -357,6 +386,14 @@ moe_gemm_kernel(const TA* A, int64_t lda, int a_div, const TW* __restrict__ Wt, 
   for (int i = 0; i < 2; ++i) {
     const int p = rows[ty * 2 + i];
     if (p < 0) continue;
+    if (act & MOE_GLU) {
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n + 1 < N) moe_st(out + (int64_t)p * (N / 2) + n / 2, moe_act(acc[i][j], act & ~MOE_GLU) * acc[i][j + 1]);
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
@@ -439,6 +476,18 @@ moe_gemv_kernel(const __nv_bfloat16* A, int64_t lda, int a_div, const __nv_bfloa
     __syncthreads();
   }
   if (n0 >= N) return;
+  if (act & MOE_GLU) {
+#pragma unroll
+    for (int f = 0; f < MV_FEAT; f += 2)
+#pragma unroll
+      for (int r = 0; r < MV_ROWS; ++r) {
+        const float g = warp_sum(acc[f][r]), u = warp_sum(acc[f + 1][r]);
+        const int p = rows[r];
+        if (lane == 0 && p >= 0 && n0 + f + 1 < N)
+          moe_st(out + (int64_t)p * (N / 2) + (n0 + f) / 2, moe_act(g, act & ~MOE_GLU) * u);
+      }
+    return;
+  }
 #pragma unroll
   for (int f = 0; f < MV_FEAT; ++f)
 #pragma unroll
@@ -682,6 +731,31 @@ extern "C" int exl3_moe_plan(const int* idx, int P, int n_experts, int tile_rows
   return launch_status("moe_plan");
 }
 
+extern "C" int exl3_moe_table_plans(const int* ids, int T, int n_layers, const int* const* tables, const int* top,
+                                    const int* n_experts, const int* tile_rows, int* const* order, int* const* plan,
+                                    cudaStream_t stream) {
+  if (T == 0 || n_layers == 0) return 0;
+  if (T < 0 || n_layers < 0) { set_error("moe_table_plans: bad sizes"); return ERR_BAD_ARGUMENT; }
+  for (int l0 = 0; l0 < n_layers; l0 += MOE_TABLES) {
+    const int n = n_layers - l0 < MOE_TABLES ? n_layers - l0 : MOE_TABLES;
+    MoeTables m = {};
+    int most = 0;
+    for (int l = 0; l < n; ++l) {
+      if (top[l0 + l] < 1 || n_experts[l0 + l] < 1 || n_experts[l0 + l] > 4096 || tile_rows[l0 + l] < 1) {
+        set_error("moe_table_plans: bad sizes of layer %d: top=%d experts=%d", l0 + l, top[l0 + l], n_experts[l0 + l]);
+        return ERR_BAD_ARGUMENT;
+      }
+      m.table[l] = tables[l0 + l]; m.order[l] = order[l0 + l]; m.plan[l] = plan[l0 + l];
+      m.top[l] = top[l0 + l]; m.n_experts[l] = n_experts[l0 + l]; m.tile_rows[l] = tile_rows[l0 + l];
+      if (m.n_experts[l] > most) most = m.n_experts[l];
+    }
+    launch_pdl(moe_table_plans_kernel, dim3(n), dim3(1024), (size_t)3 * most * sizeof(int), stream, ids, T, m);
+    const int rc = launch_status("moe_table_plans");
+    if (rc) return rc;
+  }
+  return 0;
+}
+
 // The most tiles of at most tile_rows rows that a step of P pairs over n_experts experts can have.
 extern "C" int exl3_moe_max_tiles(int P, int n_experts, int tile_rows) {
   return tile_rows < 1 ? 0 : min(P, P / tile_rows + n_experts);
@@ -700,7 +774,7 @@ extern "C" int exl3_moe_gemm(const void* A, int a_dtype, int64_t lda, int a_div,
                              const int* order, const int* plan, void* out, int out_dtype, int P, int n_experts, int N,
                              int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || N < 1 || K < 1 || a_div < 1 || act < 0 || act > 4) {
+  if (P < 0 || n_experts < 1 || N < 1 || K < 1 || a_div < 1 || act < 0 || (act & ~MOE_GLU) > 4 || ((act & MOE_GLU) && N % 2 != 0)) {
     set_error("moe_gemm: bad sizes pairs=%d experts=%d N=%d K=%d", P, n_experts, N, K);
     return ERR_BAD_ARGUMENT;
   }
@@ -725,8 +799,8 @@ extern "C" int exl3_moe_gemv_rows() { return MV_ROWS; }
 extern "C" int exl3_moe_gemv(const void* A, int64_t lda, int a_div, const void* W, const int* order, const int* plan,
                              void* out, int out_dtype, int P, int n_experts, int N, int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || N < 1 || K < 8 || K % 8 != 0 || lda % 8 != 0 || a_div < 1 || act < 0 || act > 4 ||
-      !aligned16(A) || !aligned16(W)) {
+  if (P < 0 || n_experts < 1 || N < 1 || K < 8 || K % 8 != 0 || lda % 8 != 0 || a_div < 1 || act < 0 || (act & ~MOE_GLU) > 4 ||
+      ((act & MOE_GLU) && N % 2 != 0) || !aligned16(A) || !aligned16(W)) {
     set_error("moe_gemv: bad sizes pairs=%d experts=%d N=%d K=%d (K and the row pitch multiples of 8, 16-byte aligned)", P,
               n_experts, N, K);
     return ERR_BAD_ARGUMENT;

@@ -13,7 +13,7 @@
 //   warp 0    TMA producer: 128 x 64 boxes of A and 256 x 64 boxes of W into a ring of four 128B-swizzled stages
 //   warp 1    one thread issues tcgen05.mma (M 128, N 256, K 16); tcgen05.commit frees stages and hands over accumulators
 //   warps 2-5 epilogue: thread = row, 32 accumulator columns at a time from tensor memory, the activation, and
-//             16-byte stores: in the plan's order (the first projection's output, the second one's input) or to the
+//             (with the GLU bit of act, act(even column) * (odd column)), 16-byte stores: in the plan's order (the first projection's output, the second one's input) or to the
 //             pair's own place order[i] (float32, for the weighted sum)
 // Two accumulators let the epilogue of one tile overlap the products of the next.  Work items are dealt to the blocks in turn
 // with the plan's tile fastest: blocks that run together read the same 256 rows of an expert that has several tiles.
@@ -45,6 +45,7 @@ __device__ inline float mt_act(float v, int act) {
   if (act == 4) { const float r = fmaxf(v, 0.0f); return r * r; }
   return v;
 }
+constexpr int MT_GLU = 16;                      // as moe.cu's MOE_GLU
 
 __device__ inline void mt_store8(__nv_bfloat16* p, const float (&v)[8]) { store_vec(p, v); }
 __device__ inline void mt_store8(float* p, const float (&v)[8]) {
@@ -160,6 +161,20 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
         tmem_ld32(taddr + c * 32, v);
         const int col = n0 + c * 32;
         if (!row_ok || col >= N) continue;
+        if (act & MT_GLU) {                      // 16 columns make 8 outputs
+          TO* dst = out + dst_row * (N / 2) + col / 2;
+#pragma unroll
+          for (int p = 0; p < 2; ++p) {
+            if (col + p * 16 + 16 <= N) {
+              float o8[8];
+#pragma unroll
+              for (int j = 0; j < 8; ++j)
+                o8[j] = mt_act(__uint_as_float(v[p * 16 + 2 * j]), act & ~MT_GLU) * __uint_as_float(v[p * 16 + 2 * j + 1]);
+              mt_store8(dst + p * 8, o8);
+            }
+          }
+          continue;
+        }
         TO* dst = out + dst_row * N + col;
 #pragma unroll
         for (int p = 0; p < 4; ++p) {
@@ -215,7 +230,7 @@ extern "C" int exl3_moe_tc_supported(int N, int K) { return N >= 8 && N % 8 == 0
 extern "C" int exl3_moe_gemm_tc(const void* A, const void* W, const int* order, const int* plan, void* out, int out_dtype,
                                 int P, int n_experts, int N, int K, int act, cudaStream_t stream) {
   if (P == 0) return 0;
-  if (P < 0 || n_experts < 1 || !exl3_moe_tc_supported(N, K) || act < 0 || act > 4 ||
+  if (P < 0 || n_experts < 1 || !exl3_moe_tc_supported(N, K) || act < 0 || (act & ~MT_GLU) > 4 || ((act & MT_GLU) && N % 16 != 0) ||
       (out_dtype != DT_BF16 && out_dtype != DT_F32)) {
     set_error("moe_gemm_tc: needs N and K multiples of 8 and a bfloat16 or float32 output, got pairs=%d experts=%d N=%d "
               "K=%d out=%d", P, n_experts, N, K, out_dtype);

@@ -6,6 +6,8 @@
 //   rotary encoding of the first `rot` features at the token's position p, angle a_i = p f_i:
 //       layout 0 pairs feature i with i + rot / 2, layout 1 feature 2i with 2i + 1;
 //       (u, v) <- (u cos a - v sin a, v cos a + u sin a), sines and cosines times mscale
+//   gates (g_off >= 0): gate_out[t, h] = 1 / (1 + exp(-x[t, g_off + h])), a float32 factor per query head for the
+//   attention kernel to multiply its output by
 //   keys times k_mul; queries times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)   (temp_every 0: as they are)
 //   values: v <- (1 - lambda) v + lambda v_src   when a mixing weight is given (v_src: another layer's values of
 //       the same token)
@@ -45,7 +47,15 @@ struct QkPrepArgs {
   const void* lambda; int lambda_dtype; const void* v_src; int v_src_dtype; int64_t v_src_ld;
   const int* tok_pos; const int* tok_seq; const int* block_table; int bt_stride, page;
   void* q_out; int q_out_dtype; void* k_out; int k_out_dtype; void* k_pool; void* v_pool; int pool_dtype;
+  int g_off; float* gate_out;
 };
+
+// The token's gates, by the blocks that take its first heads.
+__device__ inline void qp_gates(const QkPrepArgs& a, int t) {
+  if (a.gate_out == nullptr || blockIdx.y != 0) return;
+  for (int h = threadIdx.x; h < a.nh; h += blockDim.x)
+    a.gate_out[(int64_t)t * a.nh + h] = 1.0f / (1.0f + expf(-qp_load_act(a.x, a.x_dtype, (int64_t)t * a.ld + a.g_off + h)));
+}
 
 // What a query is multiplied by at position pos.  The quotient of two float32 numbers is rounded correctly, so its floor
 // is right for every position below 2^24.
@@ -70,6 +80,7 @@ __global__ void __launch_bounds__(QP_WARPS * 32) qk_prep_kernel(QkPrepArgs a, in
   if (a.k_pool != nullptr)
     pg = __ldcg(a.block_table + (int64_t)__ldcg(a.tok_seq + t) * a.bt_stride + pos / a.page);
   const int in_page = a.k_pool != nullptr ? pos % a.page : 0;
+  qp_gates(a, t);
   const int jobs = a.nh + a.nkv + (a.v_off >= 0 ? a.nkv : 0);
   const float q_mul = qp_temperature(a, pos);
   const float fpos = (float)pos;
@@ -216,6 +227,7 @@ __global__ void __launch_bounds__(QP_WARPS * 32) qk_prep_vec_kernel(QkPrepArgs a
   const int pos = __ldcg(a.tok_pos + t);
   const int pg = a.nkv > 0 ? __ldcg(a.block_table + (int64_t)__ldcg(a.tok_seq + t) * a.bt_stride + pos / a.page) : -1;
   const int in_page = a.nkv > 0 ? pos % a.page : 0;
+  qp_gates(a, t);
   const int half = a.rot >> 1;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, cs;
@@ -327,13 +339,14 @@ extern "C" int exl3_qk_prep(const void* x, int x_dtype, int64_t ld, int q_off, i
                             int lambda_dtype, const void* v_src, int v_src_dtype, int64_t v_src_ld, const int* tok_pos,
                             const int* tok_seq, const int* block_table, int bt_stride, int page, void* q_out,
                             int q_out_dtype, void* k_out, int k_out_dtype, void* k_pool, void* v_pool, int pool_dtype,
-                            float temp_coef, float temp_every, cudaStream_t stream) {
+                            float temp_coef, float temp_every, int g_off, float* gate_out, cudaStream_t stream) {
   if (T == 0) return 0;
   if (T < 0 || nh < 1 || nkv < 0 || hd < 1 || hd_pad < hd || (v_off >= 0 && (hdv < 1 || hdv_pad < hdv)) ||
       norm < 0 || norm > 3 || !(temp_every >= 0.0f) || rot < 0 || rot > hd || rot % 2 != 0 || layout < 0 || layout > 1 ||
       (rot > 0 && inv_freq == nullptr) || (norm >= 2 && (q_w == nullptr || (nkv > 0 && k_w == nullptr))) || q_out == nullptr ||
       (nkv > 0 && k_pool == nullptr && k_out == nullptr) || (nkv == 0 && (k_pool != nullptr || v_off >= 0)) || (k_pool != nullptr && (block_table == nullptr || page < 1)) ||
-      (v_off >= 0 && k_pool != nullptr && v_pool == nullptr) || (mix_lambda != nullptr && v_src == nullptr)) {
+      (v_off >= 0 && k_pool != nullptr && v_pool == nullptr) || (mix_lambda != nullptr && v_src == nullptr) ||
+      (gate_out != nullptr && g_off < 0)) {
     set_error("qk_prep: bad arguments T=%d heads=%d/%d head_dim=%d (%d) value_dim=%d (%d) norm=%d rot=%d layout=%d",
               T, nh, nkv, hd, hd_pad, hdv, hdv_pad, norm, rot, layout);
     return ERR_BAD_ARGUMENT;
@@ -346,6 +359,7 @@ extern "C" int exl3_qk_prep(const void* x, int x_dtype, int64_t ld, int q_off, i
   a.lambda = mix_lambda; a.lambda_dtype = lambda_dtype; a.v_src = v_src; a.v_src_dtype = v_src_dtype;
   a.v_src_ld = v_src_ld;
   a.tok_pos = tok_pos; a.tok_seq = tok_seq; a.block_table = block_table; a.bt_stride = bt_stride; a.page = page;
+  a.g_off = g_off; a.gate_out = gate_out;
   a.q_out = q_out; a.q_out_dtype = q_out_dtype; a.k_out = k_out; a.k_out_dtype = k_out_dtype;
   a.k_pool = k_pool; a.v_pool = v_pool; a.pool_dtype = pool_dtype;
   // the common case with 16-byte accesses (see qk_prep_vec_kernel)

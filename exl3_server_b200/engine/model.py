@@ -13,6 +13,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..cache.kv import SequenceCache
+from ..ops import kernels as K
 from ..parts.base import BuildContext, KVRequest, StateRequest
 from ..parts.registry import (arrangement_class, embedding_class, feed_forward_class, head_class, mixer_class,
                               norm_class)
@@ -36,15 +37,30 @@ def plan_manifest(plan: ModelPlan) -> List[TensorSpec]:
         if layer.feed_forward is not None:
             specs += feed_forward_class(layer.feed_forward.kind).tensor_specs(layer.feed_forward,
                                                                              layer.names["feed_forward"])
-            specs += norm_class(layer.feed_forward_norm.kind).tensor_specs(layer.feed_forward_norm,
-                                                                          layer.names["feed_forward_norm"])
+            if layer.feed_forward_norm is not None:             # none where both sublayers read one norm's output
+                specs += norm_class(layer.feed_forward_norm.kind).tensor_specs(layer.feed_forward_norm,
+                                                                              layer.names["feed_forward_norm"])
     for layer in plan.layers:
         arrangement = arrangement_class(layer.arrangement)
         if hasattr(arrangement, "tensor_specs"):            # arrangements with tensors of their own (layer scales)
             specs += arrangement.tensor_specs(layer)
+    if plan.entry_vectors is not None:
+        specs.append(TensorSpec(plan.entry_vectors[0], (plan.entry_vectors[1], plan.embedding.width)))
     specs += norm_class(plan.final_norm.kind).tensor_specs(plan.final_norm, plan.final_norm_name)
     specs += head_class(plan.head.kind).tensor_specs(plan.head)
     return specs
+
+
+def enter(stream, entry, block) -> None:
+    """Adds an entry's terms to the residual in a kernel of their own (where no block before has done it), with the block's
+    first norm where that is a single RMS norm."""
+    y, s = stream.take()
+    norms = block.input_norms() if hasattr(block, "input_norms") else ()
+    fused = len(norms) == 1 and hasattr(norms[0], "rms_args")
+    x = K.residual_step(stream.h, y, scale=s, entry=entry, norm=norms[0].rms_args() if fused else None)
+    stream.act = stream.normed = None
+    if fused:
+        stream.leave_for(norms, [x])
 
 
 class Model:
@@ -63,8 +79,9 @@ class Model:
             if layer.feed_forward is not None:
                 ff = feed_forward_class(layer.feed_forward.kind)(layer.feed_forward, tensors,
                                                                  layer.names["feed_forward"], ctx)
-                n2 = norm_class(layer.feed_forward_norm.kind)(layer.feed_forward_norm, tensors,
-                                                              layer.names["feed_forward_norm"], ctx)
+                if layer.feed_forward_norm is not None:
+                    n2 = norm_class(layer.feed_forward_norm.kind)(layer.feed_forward_norm, tensors,
+                                                                  layer.names["feed_forward_norm"], ctx)
             if layer.mixer_out_norm is not None or layer.feed_forward_out_norm is not None:
                 outs = [None, None]
                 if layer.mixer_out_norm is not None:
@@ -81,6 +98,10 @@ class Model:
         self.final_norm = norm_class(plan.final_norm.kind)(plan.final_norm, tensors, plan.final_norm_name, ctx)
         self.head = head_class(plan.head.kind)(plan.head, tensors, self.embedding, ctx)
         self.vocab = plan.head.vocab
+        self.entry_vectors = None
+        if plan.entry_vectors is not None:
+            self.entry_vectors = tensors[plan.entry_vectors[0]].float().contiguous()
+        self._adds_embedding = any(e.add_embedding for e in plan.schedule)
 
     def cache_requests(self) -> List[Tuple[Optional[KVRequest], Optional[StateRequest], Optional[int]]]:
         out = []
@@ -106,22 +127,48 @@ class Model:
         else:
             stream = self.embedding.forward(batch.token_ids)
         sched = self.plan.schedule
+        source = self._embedding_source(batch, stream) if self._adds_embedding else None
         for i, e in enumerate(sched):
             block = self.blocks[e.layer]
             kv, state = cache.view(i, batch.block_tables), cache.state_of(i)
+            nxt = self.blocks[sched[i + 1].layer] if i + 1 < len(sched) else None
+            entry = self._entry(i, source)
+            if entry is not None and not stream.entered:
+                enter(stream, entry, block)
+            stream.entered = False
+            coming = self._entry(i + 1, source) if nxt is not None else None
+            if coming is not None and not getattr(block, "takes_entry", False):
+                nxt = None                       # the next block's norms are over a residual that this block does not see
             if getattr(block, "takes_next", False):
-                # the block that runs next, so that this block's last kernel may also apply that block's first norms
-                block.forward(stream, batch, kv, state,
-                              next_block=self.blocks[sched[i + 1].layer] if i + 1 < len(sched) else None)
+                # the block that runs next, so that this block's last kernel may also apply that block's first norms; a
+                # block that takes entries also adds what joins the residual in between (and sets stream.entered)
+                extra = {"entry": coming} if getattr(block, "takes_entry", False) else {}
+                block.forward(stream, batch, kv, state, next_block=nxt, **extra)
             elif getattr(block, "takes_after", False):
                 # the norm that the next block applies first, so that this block's last projection may apply it
-                nxt = self.blocks[sched[i + 1].layer] if i + 1 < len(sched) else None
                 block.forward(stream, batch, kv, state, after=getattr(nxt, "mixer_norm", None))
             else:
                 block.forward(stream, batch, kv, state)
         if batch.n_wanted == 0:
             return None
         return self.head.forward(stream, self.final_norm, batch.want_rows)
+
+    def _embedding_source(self, batch: StepBatch, stream):
+        """``(rows, ids, scale)`` from which the embedding's output can be read again: its table where the embedding is a
+        row of it, else a copy of the residual as it stands now."""
+        rows = getattr(self.embedding, "row_source", None)
+        if rows is not None:
+            table, scale = rows()
+            return table, batch.token_ids, scale
+        return stream.h.clone(), None, 1.0
+
+    def _entry(self, i: int, source):
+        """What joins the residual ahead of schedule entry i, as ``kernels.residual_step`` takes it, or None."""
+        e = self.plan.schedule[i]
+        if not e.add_embedding and e.add_vector is None:
+            return None
+        emb, ids, scale = source if e.add_embedding else (None, None, 0.0)
+        return emb, ids, scale, self.entry_vectors[e.add_vector] if e.add_vector is not None else None
 
     def weight_bytes(self, tokens: Optional[int] = None) -> int:
         """Bytes of weights that one step reads (each matrix once; a tied head

@@ -522,18 +522,20 @@ def attn_tokens_ex(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool
                    T: int, heads: int, kv_heads: int, head_dim: int, value_dim: int, page: int, window: int,
                    chunk: int, sink: bool, scale: float, split_keys: int, max_splits: int,
                    scratch: Optional[torch.Tensor], keep_first: int = 0, softcap: float = 0.0,
-                   sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                   gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``attn_tokens`` in its general form: rows of the key pool hold ``head_dim`` features and rows of the value
     pool ``value_dim`` (each pool's last dimension is its row pitch; multiples of 8; values may be wider than keys);
     ``chunk`` > 0 also hides every key before ``floor(pos / chunk) * chunk``; ``sink`` adds one to the softmax's
     denominator (``sink_vals`` float32 ``[heads]``: ``exp`` of a score per head instead of one).  With a window,
     keys at positions below ``keep_first`` stay visible (``max_splits`` then counts their chunks too); ``softcap``
     > 0 caps the scaled scores, ``c tanh(s / c)``; ``dist`` (a ``distance_table``) adds a bias per head and distance to
-    them.  ``out`` is ``[T, heads, value_dim]`` in the cache's type or
+    them; ``gate`` (float32 ``[T, heads]``) is a factor per token and head on the output.  ``out`` is ``[T, heads, value_dim]`` in the cache's type or
     float32 (for callers that go on in float32) and the scratch is sized with ``value_dim``."""
     if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
         raise KernelLibraryError("attn_tokens_ex: sink scores must be float32 [heads], with the sink on")
     dist_len = _distance_len(dist, heads, "attn_tokens_ex")
+    _check_gate(gate, T, heads, "attn_tokens_ex")
     if k_pool.dtype != q.dtype or v_pool.dtype != q.dtype or out.dtype not in (q.dtype, torch.float32):
         raise KernelLibraryError("attn_tokens_ex: q, cache and out differ in element type")
     nbytes = 0 if scratch is None else scratch.numel() * scratch.element_size()
@@ -544,7 +546,7 @@ def attn_tokens_ex(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool
         _c_int(heads), _c_int(kv_heads), _c_int(head_dim), _c_int(value_dim), _c_int(k_pool.shape[-1]),
         _c_int(v_pool.shape[-1]), _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0),
         _c_float(scale), _c_int(split_keys), _c_int(max_splits), _ptr(scratch), _c_size_t(nbytes), _c_int(keep_first),
-        _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()), "attn_tokens_ex")
+        _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _ptr(gate), _stream()), "attn_tokens_ex")
     return out
 
 
@@ -564,6 +566,11 @@ def _distance_len(dist: Optional[torch.Tensor], heads: int, what: str) -> int:
             not dist.is_contiguous():
         raise KernelLibraryError(f"{what}: distance biases must be a contiguous float32 distance_table with a row per head")
     return dist.shape[1] - 2 * DIST_PAD
+
+
+def _check_gate(gate: Optional[torch.Tensor], T: int, heads: int, what: str) -> None:
+    if gate is not None and (gate.dtype != torch.float32 or gate.numel() != T * heads or not gate.is_contiguous()):
+        raise KernelLibraryError(f"{what}: the output's factors must be float32 [tokens, heads]")
 
 
 def embed_sinusoid(ids: torch.Tensor, tok_pos: torch.Tensor, table: torch.Tensor, scale: float, frequencies: torch.Tensor,
@@ -617,12 +624,14 @@ def qk_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_
             mscale: float, k_mul: float, mix: Optional[tuple], tok_pos: torch.Tensor, tok_seq: torch.Tensor,
             block_table: Optional[torch.Tensor], page: int, q_dtype: torch.dtype,
             k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
-            k_dtype: Optional[torch.dtype] = None, temperature: Optional[tuple] = None):
+            k_dtype: Optional[torch.dtype] = None, temperature: Optional[tuple] = None,
+            gate_off: Optional[int] = None):
     """Norm, rotation, value mixing and the cache write between an attention's joint projection ``x [T, ld]`` and
     the attention (see qk_prep.cu).  ``mix``: ``(lambda tensor, v_src [T, *] view)`` or None.  Returns ``(q, k)``:
     the queries ``[T, heads * head_pad]`` and, when there is no ``k_pool``, the keys ``[T, kv_heads * head_pad]``
     (else None).  ``kv_heads`` 0: queries only (``v_off`` -1, no pools).  ``temperature``: ``(coef, every)``; queries at
-    position p are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
+    position p are multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``gate_off``: the columns from there on hold a gate's
+    logit per query head; their sigmoids come back as a third result, float32 ``[T, heads]``."""
     T = x.shape[0]
     if x.stride(1) != 1:
         raise KernelLibraryError("qk_prep: rows of x must be dense")
@@ -632,6 +641,7 @@ def qk_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_
     if k_pool is None and kv_heads > 0:
         k = torch.empty((T, kv_heads * head_pad), dtype=k_dtype or q_dtype, device=x.device)
     lam, v_src = mix if mix is not None else (None, None)
+    gate = torch.empty((T, heads), dtype=torch.float32, device=x.device) if gate_off is not None else None
     if v_src is not None and v_src.stride(1) != 1:
         raise KernelLibraryError("qk_prep: rows of the mixed-in values must be dense")
     _check(library().exl3_qk_prep(
@@ -645,9 +655,9 @@ def qk_prep(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_
         _c_int(block_table.stride(0) if block_table is not None else 0), _c_int(page), _ptr(q),
         _c_int(dtype_code(q.dtype)), _ptr(k), _c_int(dtype_code(k.dtype) if k is not None else 0), _ptr(k_pool),
         _ptr(v_pool), _c_int(dtype_code(k_pool.dtype) if k_pool is not None else 0),
-        _c_float(temperature[0] if temperature else 0.0), _c_float(temperature[1] if temperature else 0.0), _stream()),
-        "qk_prep")
-    return q, k
+        _c_float(temperature[0] if temperature else 0.0), _c_float(temperature[1] if temperature else 0.0),
+        _c_int(gate_off if gate_off is not None else -1), _ptr(gate), _stream()), "qk_prep")
+    return (q, k) if gate_off is None else (q, k, gate)
 
 
 def token_shift(h: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, tok_seq: torch.Tensor, row_start: torch.Tensor,
@@ -899,22 +909,23 @@ def mingru_scan(zug: torch.Tensor, state: torch.Tensor, slot_ids: torch.Tensor, 
 def latent_prep(a: torch.Tensor, q_off: int, q_rank: int, wq: torch.Tensor, kv_off: int, kv_rank: int, rot_dim: int,
                 wkv: Optional[torch.Tensor], g_off: int, heads: int, eps: float, inv_freq: Optional[torch.Tensor],
                 rot: int, tok_pos: torch.Tensor, tok_seq: torch.Tensor, block_table: torch.Tensor, page: int,
-                pool: Optional[torch.Tensor], kv_row: int, rank_pad: int, cq_dtype: torch.dtype):
+                pool: Optional[torch.Tensor], kv_row: int, rank_pad: int, cq_dtype: torch.dtype, layout: int = 0,
+                mscale: float = 1.0):
     """Latent attention's step between the joint input projection ``a`` and the rest (see latent.cu): returns the
-    normed query latent ``[T, q_rank]`` and the float32 gates ``[T, heads]``; writes each token's row of the cache
-    (``pool``; None for a layer that reads another layer's rows)."""
+    normed query latent ``[T, q_rank]`` and the float32 gates ``[T, heads]`` (None with ``heads`` 0); writes each token's row
+    of the cache (``pool``; None for a layer that reads another layer's rows).  ``layout`` and ``mscale`` as in ``qk_prep``."""
     T = a.shape[0]
     _contig(a, "a")
     f_hi, f_lo = (_rotary_rows(inv_freq, rot, "latent_prep") if rot > 0 and inv_freq is not None
                   else (_c_void_p(0), _c_void_p(0)))
     cq = torch.empty((T, q_rank), dtype=cq_dtype, device=a.device)
-    gate = torch.empty((T, heads), dtype=torch.float32, device=a.device)
+    gate = torch.empty((T, heads), dtype=torch.float32, device=a.device) if heads else None
     _check(library().exl3_latent_prep(
         _ptr(a), _c_int(dtype_code(a.dtype)), _c_int(a.shape[1]), _c_int(T), _c_int(q_off), _c_int(q_rank), _ptr(wq),
         _c_int(dtype_code(wq.dtype)), _c_int(kv_off), _c_int(kv_rank), _c_int(rot_dim), _ptr(wkv),
         _c_int(dtype_code(wkv.dtype) if wkv is not None else 0), _c_int(g_off), _c_int(heads), _c_float(eps), f_hi, f_lo,
-        _c_int(rot), _ptr(tok_pos), _ptr(tok_seq), _ptr(block_table), _c_int(block_table.stride(0)), _c_int(page),
-        _ptr(pool), _c_int(dtype_code(pool.dtype) if pool is not None else 0), _c_int(kv_row), _c_int(rank_pad),
+        _c_int(rot), _c_int(layout), _c_float(mscale), _ptr(tok_pos), _ptr(tok_seq), _ptr(block_table),
+        _c_int(block_table.stride(0)), _c_int(page), _ptr(pool), _c_int(dtype_code(pool.dtype) if pool is not None else 0), _c_int(kv_row), _c_int(rank_pad),
         _ptr(cq), _c_int(dtype_code(cq.dtype)), _ptr(gate), _stream()), "latent_prep")
     return cq, gate
 
@@ -922,10 +933,13 @@ def latent_prep(a: torch.Tensor, q_off: int, q_rank: int, wq: torch.Tensor, kv_o
 def head_gemm(x: torch.Tensor, x_row: int, x_head: int, w: Optional[torch.Tensor], out: torch.Tensor, out_row: int,
               out_head: int, T: int, heads: int, K: int, N: int, mul: Optional[torch.Tensor] = None, rot_dim: int = 0,
               rot: int = 0, inv_freq: Optional[torch.Tensor] = None, tok_pos: Optional[torch.Tensor] = None,
-              tail_off: int = 0) -> torch.Tensor:
+              tail_off: int = 0, layout: int = 0, mscale: float = 1.0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[t, h, n] = mul[t, h] * sum_k x[t, h, k] w[h, k, n]`` with the given row and head pitches (elements);
     with ``rot_dim`` the features behind a head's ``K`` are rotated and written at ``tail_off`` (see latent.cu).  With
-    ``w`` None only those tails (and the zeros around them) are written."""
+    ``w`` None only those tails (and the zeros around them) are written.  ``gate`` ``[T, heads * N]`` (any row pitch): logits
+    whose sigmoids are one more factor of the outputs."""
+    if gate is not None and (gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * N)):
+        raise KernelLibraryError("head_gemm: the gate must be [T, heads * N] with dense rows")
     if w is not None:
         if w.dtype != x.dtype or tuple(w.shape) != (heads, K, N):
             raise KernelLibraryError(f"head_gemm: w {tuple(w.shape)} must be {(heads, K, N)} in the type of x and out")
@@ -936,9 +950,22 @@ def head_gemm(x: torch.Tensor, x_row: int, x_head: int, w: Optional[torch.Tensor
                   else (_c_void_p(0), _c_void_p(0)))
     _check(library().exl3_head_gemm(
         _ptr(x), _c_int64(x_row), _c_int(x_head), _ptr(w), _ptr(out), _c_int64(out_row), _c_int(out_head),
-        _c_int(dtype_code(x.dtype)), _c_int(T), _c_int(heads), _c_int(K), _c_int(N), _ptr(mul), _c_int(rot_dim),
-        _c_int(rot), f_hi, f_lo, _ptr(tok_pos), _c_int(tail_off), _stream()), "head_gemm")
+        _c_int(dtype_code(x.dtype)), _c_int(T), _c_int(heads), _c_int(K), _c_int(N), _ptr(mul), _ptr(gate),
+        _c_int(dtype_code(gate.dtype) if gate is not None else 0), _c_int64(gate.stride(0) if gate is not None else 0),
+        _c_int(rot_dim), _c_int(rot), _c_int(layout), _c_float(mscale), f_hi, f_lo, _ptr(tok_pos), _c_int(tail_off),
+        _stream()), "head_gemm")
     return out
+
+
+def sigmoid_mul(y: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``y *= sigmoid(gate)`` in place: ``y [T, n]``, ``gate [T, n]`` with any row pitch; float32 inside."""
+    _contig(y, "y")
+    if gate.shape != y.shape or gate.stride(1) != 1:
+        raise KernelLibraryError("sigmoid_mul: the gate must be as large as y, with dense rows")
+    _check(library().exl3_sigmoid_mul(_ptr(y), _c_int(dtype_code(y.dtype)), _ptr(gate), _c_int(dtype_code(gate.dtype)),
+                                      _c_int64(gate.stride(0)), _c_int(y.shape[0]), _c_int(y.shape[1]), _stream()),
+           "sigmoid_mul")
+    return y
 
 
 def attn_prefill_tc_supported(dtype: torch.dtype, head_dim: int, page: int) -> bool:
@@ -955,14 +982,16 @@ def attn_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
                     tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, heads: int, kv_heads: int,
                     head_dim: int, page: int, window: int, scale: float, variant: int = 0, chunk: int = 0,
                     sink: bool = False, keep_first: int = 0, softcap: float = 0.0,
-                    sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of whole prompts on tcgen05 tensor cores (tiles of 128 queries; see
     attention_prefill_tc.cu).  ``k_pool`` / ``v_pool``: one layer's ``[pages, kv_heads, 64, head_dim]``.
     ``variant``: 0 lets the kernel choose by the number of blocks between a tile a block, four blocks per SM (heads
     of 64) and two tiles a block (the list's first with its last, and so on: list the tiles with the most keys
     to visit first); 1, 2 and 3 force one of them (the same numbers every way).  ``chunk``, ``sink``, ``keep_first``,
-    ``softcap``, ``sink_vals`` and ``dist`` as in ``attn_tokens_ex``."""
+    ``softcap``, ``sink_vals``, ``dist`` and ``gate`` as in ``attn_tokens_ex``."""
     dist_len = _distance_len(dist, heads, "attn_prefill_tc")
+    _check_gate(gate, q.shape[0], heads, "attn_prefill_tc")
     if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
         raise KernelLibraryError("attn_prefill_tc: sink scores must be float32 [heads], with the sink on")
     if k_pool.dtype != q.dtype or v_pool.dtype != q.dtype or out.dtype != q.dtype:
@@ -975,7 +1004,7 @@ def attn_prefill_tc(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
         _c_int64(pool_rows), _ptr(block_table), _c_int(block_table.stride(0)), _ptr(row_start), _ptr(row_pos0),
         _ptr(tile_seq), _ptr(tile_q0), _c_int(n_tiles), _c_int(heads), _c_int(kv_heads), _c_int(head_dim),
         _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0), _c_float(scale), _c_int(variant),
-        _c_int(keep_first), _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()),
+        _c_int(keep_first), _c_float(softcap), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _ptr(gate), _stream()),
         "attn_prefill_tc")
     return out
 
@@ -1013,7 +1042,8 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
                 max_splits: int, scratch: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor] = None,
                 rot: int = 0, pos_scale: float = 1.0, write_new: bool = False, head_split: int = 1,
                 in_block: int = 0, twins: int = 1, chunk: int = 0, sink: bool = False,
-                sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None) -> torch.Tensor:
+                sink_vals: Optional[torch.Tensor] = None, dist: Optional[torch.Tensor] = None,
+                gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of T query tokens over the paged cache on the tensor cores (see attention_decode.cu);
     arguments and scratch as ``attn_tokens``.  With ``write_new``, ``q`` is the fused q|k|v output of the
     projection, every token is its sequence's only new one and the cache holds the positions before it: the
@@ -1027,7 +1057,8 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
     tickets; results differ from the other way's by rounding (another order of the same sums).  ``twins`` 2 (with
     ``in_block`` 1 or 2, an even ``head_split`` and groups of up to 8 heads): a block takes two groups of query heads
     of a kv head, whose warps walk the same pages out of the same rings; changes no result.  ``chunk``, ``sink``,
-    ``sink_vals`` and ``dist`` as in ``attn_tokens_ex``."""
+    ``sink_vals``, ``dist`` and ``gate`` as in ``attn_tokens_ex``."""
+    _check_gate(gate, T, heads, "attn_decode")
     if sink_vals is not None and (sink_vals.dtype != torch.float32 or sink_vals.numel() != heads or not sink):
         raise KernelLibraryError("attn_decode: sink scores must be float32 [heads], with the sink on")
     dist_len = _distance_len(dist, heads, "attn_decode")
@@ -1048,7 +1079,7 @@ def attn_decode(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_pool: t
         _c_int(kv_heads), _c_int(head_dim), _c_int(page), _c_int(window), _c_int(chunk), _c_int(1 if sink else 0),
         _c_float(scale), _c_int(split_keys), _c_int(max_splits), _ptr(scratch), _c_size_t(nbytes), hi, lo, _c_int(rot),
         _c_float(pos_scale), _c_int(1 if write_new else 0), _c_int(head_split), _c_int(int(in_block)),
-        _c_int(int(twins)), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _stream()), "attn_decode")
+        _c_int(int(twins)), _ptr(sink_vals), _ptr(dist), _c_int(dist_len), _ptr(gate), _stream()), "attn_decode")
     return out
 
 
@@ -1240,8 +1271,45 @@ def moe_plan(idx: torch.Tensor, n_experts: int, tile_rows: int = 0):
     return order, plan
 
 
+def moe_table_plans(ids: torch.Tensor, layers):
+    """The plans of several layers whose experts a table gives by token id, in one launch: ``layers`` is a list of
+    ``(table int32 [vocab, top], experts, tile_rows)``; pair ``t * top + k`` of a layer goes to expert
+    ``table[ids[t], k]``.  Returns ``[(order, plan)]`` as ``moe_plan`` does."""
+    T = ids.numel()
+    if ids.dtype != torch.int32:
+        raise KernelLibraryError("moe_table_plans: ids must be int32")
+    sizes = [(T * t.shape[1], 4 + 3 * max(1, moe_max_tiles(T * t.shape[1], e, rows))) for t, e, rows in layers]
+    up4 = lambda n: (n + 3) // 4 * 4
+    buf = torch.empty((sum(up4(a) + up4(b) for a, b in sizes),), dtype=torch.int32, device=ids.device)
+    out, at = [], 0
+    for a, b in sizes:
+        out.append((buf[at:at + a], buf[at + up4(a):at + up4(a) + b]))
+        at += up4(a) + up4(b)
+    n = len(layers)
+    for t, _, _ in layers:
+        _contig(t, "table")
+        if t.dtype != torch.int32:
+            raise KernelLibraryError("moe_table_plans: tables must be int32")
+    pointers = lambda ts: (_c_void_p * n)(*[t.data_ptr() for t in ts])
+    ints = lambda vs: (_c_int * n)(*vs)
+    _ptr(buf)
+    _check(library().exl3_moe_table_plans(
+        _ptr(ids), _c_int(T), _c_int(n), pointers([t for t, _, _ in layers]), ints([t.shape[1] for t, _, _ in layers]),
+        ints([e for _, e, _ in layers]), ints([r for _, _, r in layers]), pointers([o for o, _ in out]),
+        pointers([p for _, p in out]), _stream()), "moe_table_plans")
+    return out
+
+
+MOE_GLU = 16          # bit of the activation's code
+
+
+def _moe_act(act: str, glu: bool, N: int):
+    """(code, width of the results): with ``glu`` the experts' rows alternate between a gate's and an up projection's."""
+    return (MOE_ACTIVATIONS[act] + MOE_GLU, N // 2) if glu else (MOE_ACTIVATIONS[act], N)
+
+
 def moe_gemv(a: torch.Tensor, a_div: int, w: torch.Tensor, order: torch.Tensor, plan: torch.Tensor,
-             out_dtype: torch.dtype, act: str = "none") -> torch.Tensor:
+             out_dtype: torch.dtype, act: str = "none", glu: bool = False) -> torch.Tensor:
     """``moe_gemm`` for a plan of tiles of at most ``moe_tile_rows("few")`` rows (decode): bfloat16 ``a`` and ``w``, inputs
     a multiple of 8 wide; every expert's matrix is read once, a warp per output feature."""
     E, N, Kd = w.shape
@@ -1249,10 +1317,11 @@ def moe_gemv(a: torch.Tensor, a_div: int, w: torch.Tensor, order: torch.Tensor, 
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.stride(1) != 1 or a.shape[1] != Kd:
         raise KernelLibraryError("moe_gemv: a and w must be bfloat16, rows of a dense and as wide as the experts' inputs")
     P = order.numel()
-    out = torch.empty((P, N), dtype=out_dtype, device=a.device)
+    code, wide = _moe_act(act, glu, N)
+    out = torch.empty((P, wide), dtype=out_dtype, device=a.device)
     _check(library().exl3_moe_gemv(
         _ptr(a), _c_int64(a.stride(0)), _c_int(a_div), _ptr(w), _ptr(order), _ptr(plan), _ptr(out),
-        _c_int(dtype_code(out_dtype)), _c_int(P), _c_int(E), _c_int(N), _c_int(Kd), _c_int(MOE_ACTIVATIONS[act]),
+        _c_int(dtype_code(out_dtype)), _c_int(P), _c_int(E), _c_int(N), _c_int(Kd), _c_int(code),
         _stream()), "moe_gemv")
     return out
 
@@ -1270,7 +1339,7 @@ def moe_gather(x: torch.Tensor, top: int, order: torch.Tensor, plan: torch.Tenso
 
 
 def moe_gemm_tc(a: torch.Tensor, w: torch.Tensor, order: torch.Tensor, plan: torch.Tensor, out_dtype: torch.dtype,
-                act: str = "none") -> torch.Tensor:
+                act: str = "none", glu: bool = False) -> torch.Tensor:
     """The experts' product on tcgen05 tensor cores (see moe_tc.cu) for a plan of tiles of at most
     ``moe_tile_rows("tc")`` rows: ``a [pairs, K]`` bfloat16 in the plan's order, ``w [experts, N, K]`` bfloat16.  A bfloat16
     result is in the plan's order too; a float32 one has every pair at its own place (``order[i]``)."""
@@ -1282,28 +1351,31 @@ def moe_gemm_tc(a: torch.Tensor, w: torch.Tensor, order: torch.Tensor, plan: tor
     P = order.numel()
     if a.shape[0] != P:
         raise KernelLibraryError("moe_gemm_tc: a must have a row per pair")
-    out = torch.empty((P, N), dtype=out_dtype, device=a.device)
+    code, wide = _moe_act(act, glu, N)
+    out = torch.empty((P, wide), dtype=out_dtype, device=a.device)
     _check(library().exl3_moe_gemm_tc(
         _ptr(a), _ptr(w), _ptr(order), _ptr(plan), _ptr(out), _c_int(dtype_code(out_dtype)), _c_int(P), _c_int(E),
-        _c_int(N), _c_int(Kd), _c_int(MOE_ACTIVATIONS[act]), _stream()), "moe_gemm_tc")
+        _c_int(N), _c_int(Kd), _c_int(code), _stream()), "moe_gemm_tc")
     return out
 
 
 def moe_gemm(a: torch.Tensor, a_div: int, w: torch.Tensor, order: torch.Tensor, plan: torch.Tensor,
-             out_dtype: torch.dtype, act: str = "none") -> torch.Tensor:
+             out_dtype: torch.dtype, act: str = "none", glu: bool = False) -> torch.Tensor:
     """``out[p] = act(w[expert(p)] a[p // a_div])`` for the planned pairs: ``w [experts, N, K]``; ``a [rows, K]`` has
-    one row per pair (``a_div`` 1) or per token (``a_div`` = picks per token).  Rows of pairs that are not planned
+    one row per pair (``a_div`` 1) or per token (``a_div`` = picks per token).  ``glu``: rows 2i and 2i + 1 of an expert's
+    matrix are a gate's and an up projection's, result i is ``act(gate_i) * up_i`` and results are ``N / 2`` wide.  Rows of pairs that are not planned
     are left unwritten."""
     E, N, Kd = w.shape
     _contig(w, "w")
     if a.stride(1) != 1 or a.shape[1] != Kd:
         raise KernelLibraryError("moe_gemm: rows of a must be dense and as wide as the experts' inputs")
     P = order.numel()
-    out = torch.empty((P, N), dtype=out_dtype, device=a.device)
+    code, wide = _moe_act(act, glu, N)
+    out = torch.empty((P, wide), dtype=out_dtype, device=a.device)
     _check(library().exl3_moe_gemm(
         _ptr(a), _c_int(dtype_code(a.dtype)), _c_int64(a.stride(0)), _c_int(a_div), _ptr(w), _c_int(dtype_code(w.dtype)),
         _ptr(order), _ptr(plan), _ptr(out), _c_int(dtype_code(out_dtype)), _c_int(P), _c_int(E), _c_int(N), _c_int(Kd),
-        _c_int(MOE_ACTIVATIONS[act]), _stream()), "moe_gemm")
+        _c_int(code), _stream()), "moe_gemm")
     return out
 
 
@@ -1582,3 +1654,41 @@ def gemm_few_out(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor])
                                        _c_int(dtype_code(x.dtype)), _c_int(M), _c_int(N), _c_int(Kd), _stream()),
            "gemm_few_out")
     return out
+
+
+def residual_step(h: torch.Tensor, a: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None,
+                  picks: Optional[tuple] = None, scale: float = 1.0, entry: Optional[tuple] = None,
+                  norm: Optional[tuple] = None) -> Optional[torch.Tensor]:
+    """The residual's step between two layers, in place on ``h`` float32 ``[T, W]`` (see residual_step.cu):
+    ``h += scale * (a + b + weight * sum_k y[t, k])`` with ``picks = (y float32 [T * top, W], top, weight)``, then
+    ``h += emb_scale * emb[ids[t]] + vec`` with ``entry = (emb or None, ids or None, emb_scale, vec float32 [W] or None)``
+    (``ids`` None: row t of ``emb``).  With ``norm = (weight, eps, dtype)`` returns ``rmsnorm(h) * weight``."""
+    T, W = h.shape
+    if h.dtype != torch.float32:
+        raise KernelLibraryError("residual_step: the residual stream must be float32")
+    _contig(h, "h")
+    for n, t in (("a", a), ("b", b)):
+        if t is not None:
+            _contig(t, n)
+            if t.shape != h.shape:
+                raise KernelLibraryError(f"residual_step: {n} is {tuple(t.shape)}, h is {tuple(h.shape)}")
+    y, top, weight = picks if picks is not None else (None, 1, 0.0)
+    if y is not None:
+        _contig(y, "picks")
+        if y.dtype != torch.float32 or tuple(y.shape) != (T * top, W):
+            raise KernelLibraryError("residual_step: picks must be float32 [T * top, W]")
+    emb, ids, emb_scale, vec = entry if entry is not None else (None, None, 0.0, None)
+    if emb is not None:
+        _contig(emb, "emb")
+        if emb.shape[1] != W or (ids is None and emb.shape[0] != T) or (ids is not None and (ids.dtype != torch.int32 or ids.numel() != T)):
+            raise KernelLibraryError("residual_step: emb must be [rows, W] with int32 ids, or [T, W]")
+    if vec is not None and (vec.dtype != torch.float32 or vec.numel() != W):
+        raise KernelLibraryError("residual_step: vec must be float32 [W]")
+    w, eps, x_dtype = norm if norm is not None else (None, 0.0, torch.float32)
+    x = torch.empty((T, W), dtype=x_dtype, device=h.device) if w is not None else None
+    code = lambda t: _c_int(dtype_code(t.dtype) if t is not None else 0)
+    _check(library().exl3_residual_step(
+        _ptr(h), _ptr(a), code(a), _ptr(b), code(b), _ptr(y), _c_int(top), _c_float(weight), _c_float(scale), _ptr(emb),
+        code(emb), _ptr(ids), _c_float(emb_scale), _ptr(vec), _ptr(w), code(w), _c_float(eps), _ptr(x), code(x), _c_int(T),
+        _c_int(W), _stream()), "residual_step")
+    return x

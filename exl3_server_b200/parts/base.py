@@ -25,8 +25,8 @@ Interfaces (duck-typed; the classes below only document them):
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
-from typing import Optional, Tuple
+from dataclasses import dataclass, field
+from typing import Any, Dict, Optional, Tuple
 
 import torch
 
@@ -35,6 +35,8 @@ import torch
 class BuildContext:
     dtype: torch.dtype            # activations and matrix weights: bfloat16 or float32
     device: torch.device
+    # what parts of one model keep together (keyed as they like), such as tables that one kernel reads for all of them
+    shared: Dict[Any, Any] = field(default_factory=dict, compare=False)
 
 
 @dataclass(frozen=True)
@@ -76,6 +78,8 @@ class ResidualStream:
         # the residual as it stands in the activation type, when a block has left it (arrangements whose sublayers
         # read the residual itself); whoever changes ``h`` afterwards forgets it
         self.act: Optional[torch.Tensor] = None
+        # set by a block that has added what joins the residual ahead of the next schedule entry
+        self.entered = False
 
     def push(self, y: torch.Tensor, scale: float) -> None:
         if self.pending is not None:

@@ -21,6 +21,11 @@ float32, and the two norms that the next block of this kind applies to the new r
 vectors are tensors of the arrangement (names under ``mixer_scale`` and ``feed_forward_scale``).  A layer may have no
 feed-forward.
 
+``parallel``: both sublayers read one norm's output and their outputs are added together: with ``r = norm1(h)``,
+``h += rho * (mixer(r) + ff(r))``.  The step (float32), the sum over a routed feed-forward's picks where they have equal
+weights, what joins the residual ahead of the next layer (a schedule entry's vector and the embedding's output) and the
+next layer's norm are one kernel (``kernels.residual_step``).  A layer may have no feed-forward.
+
 ``hyper``: hyper-connections.  The residual is ``streams`` rows per token, ``x_1 .. x_S``, all equal to the embedding at
 the start.  Sublayer q (1: the mixer, 2: the feed-forward) reads ``u = sum_s a_q[s] x_s``, runs on ``norm_q(u)`` and
 writes to every stream at once from the old ones, ``x_t <- sum_s M_q[s, t] x_s + b_q[t] y`` (``M_q`` indexed [from,
@@ -204,6 +209,47 @@ class SideBySideBlock:
             (2 if self.feed_forward_scale is not None else 1)
 
 
+class ParallelBlock:
+    takes_next = True         # forward gets the block that runs next
+    takes_entry = True        # and what joins the residual ahead of it
+
+    def __init__(self, spec: LayerSpec, mixer, feed_forward, mixer_norm, feed_forward_norm):
+        if feed_forward_norm is not None:
+            raise ValueError("parallel: both sublayers read the mixer's norm")
+        self.spec = spec
+        self.mixer = mixer
+        self.feed_forward = feed_forward              # None: the layer is its mixer only
+        self.mixer_norm = mixer_norm
+        self.feed_forward_norm = None
+
+    def input_norms(self):
+        """The norms this block applies to the residual it is given."""
+        return (self.mixer_norm,)
+
+    def forward(self, stream: ResidualStream, batch, kv, state, next_block=None, entry=None) -> None:
+        left = stream.take_for(self.input_norms())
+        r = left[0] if left is not None else self.mixer_norm.add_norm(stream)
+        y = self.mixer.forward(r, batch, kv, state)
+        b = picks = None
+        if self.feed_forward is not None:
+            if hasattr(self.feed_forward, "forward_picks"):
+                picks = self.feed_forward.forward_picks(r, batch)     # the sum over the picks is the step's kernel's
+            else:
+                b = self.feed_forward.forward(r, batch)
+        nxt = next_block.input_norms() if hasattr(next_block, "input_norms") else ()
+        fused = len(nxt) == 1 and hasattr(nxt[0], "rms_args")
+        x = K.residual_step(stream.h, y, b, picks, float(self.spec.residual_scale), entry,
+                            nxt[0].rms_args() if fused else None)
+        stream.act = stream.normed = None
+        stream.entered = entry is not None
+        if fused:
+            stream.leave_for(nxt, [x])
+
+    def weight_bytes(self) -> int:
+        return sum(p.weight_bytes() for p in (self.mixer, self.feed_forward, self.mixer_norm)
+                   if p is not None and hasattr(p, "weight_bytes"))
+
+
 class HyperBlock:
     takes_tensors = True      # built with the checkpoint's tensors (read, write and mixing weights of the streams)
     takes_next = True         # forward gets the block that runs next
@@ -285,6 +331,7 @@ class HyperBlock:
 
 
 register_arrangement("prenorm", PreNormBlock)
+register_arrangement("parallel", ParallelBlock)
 register_arrangement("hyper", HyperBlock)
 register_arrangement("side_by_side", SideBySideBlock)
 register_arrangement("sandwich", SandwichBlock)

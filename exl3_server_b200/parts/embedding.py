@@ -38,6 +38,10 @@ class Embedding:
     def forward(self, token_ids: torch.Tensor) -> ResidualStream:
         return ResidualStream(K.embed(token_ids, self.table, float(self.spec.scale)))
 
+    def row_source(self):
+        """``(table, scale)``: a token's embedding is its row of the table times the scale."""
+        return self.table, float(self.spec.scale)
+
     def weight_bytes(self) -> int:
         return self.table.numel() * self.table.element_size()
 

@@ -9,6 +9,9 @@ With ``H`` heads of ``dim`` unrotated and ``rot_dim`` rotated query/key features
     s_h(i, j) = (q^n_h(i) . k^n_h(j) + rope(q^r_h(i)) . k^r(j)) * scale,   j <= i,   softmax over j
     y = concat_h( sigmoid(x wg_h) * sum_j p_h(i, j) v_h(j) ) Wo^T
 
+The gate is one number per head, or with ``gate`` ``"element"`` one per output feature (``Wg [H * vdim]``).  The rotation is
+the spec's position encoding with its pairing of features (``layout``), frequency table and factor (``yarn``, ``bands``).
+
 The cache keeps ``[c | k^r]`` per token and nothing per head.  The per-head keys and values are never formed: the
 query is carried into the latent space (``q^n_h Wuk_h``, a product per head), attention runs over the cached rows
 as keys whose leading ``kv_rank`` features are also the values, and ``Wuv_h`` is applied to what comes out.  That
@@ -60,6 +63,13 @@ class LatentAttention:
             raise ValueError(f"latent attention: sizes must be positive, got {sizes} with {spec.heads} heads")
         return sizes
 
+    @staticmethod
+    def _gate(spec: MixerSpec) -> str:
+        kind = spec.params.get("gate", "head")
+        if kind not in ("head", "element"):
+            raise ValueError(f"latent attention: gate must be 'head' or 'element', got {kind!r}")
+        return kind
+
     @classmethod
     def tensor_specs(cls, spec: MixerSpec, prefix: str) -> List[TensorSpec]:
         z = cls._sizes(spec)
@@ -70,7 +80,7 @@ class LatentAttention:
             TensorSpec(prefix + "uq", (H * (z["dim"] + z["rot_dim"]), z["q_rank"])),
             TensorSpec(prefix + "uk", (H * z["dim"], z["kv_rank"])),
             TensorSpec(prefix + "uv", (H * z["vdim"], z["kv_rank"])),
-            TensorSpec(prefix + "g", (H, spec.width)),
+            TensorSpec(prefix + "g", (H * (z["vdim"] if cls._gate(spec) == "element" else 1), spec.width)),
             TensorSpec(prefix + "o", (spec.width, H * z["vdim"])),
         ]
         if not spec.params.get("shared_rows", False):
@@ -93,8 +103,10 @@ class LatentAttention:
         if pos.dims % 2 != 0 or not 0 <= pos.dims <= self.rot_dim:
             raise ValueError(f"latent attention: {pos.dims} rotated features must be even and at most rot_dim {self.rot_dim}")
         self.rot = pos.dims
-        self.inv_freq = (K.rotary_table(RotaryPosition.frequencies(pos) * float(pos.scale)).to(ctx.device)
-                         if self.rot > 0 else None)
+        self.position = RotaryPosition(pos, self.rot_dim, ctx)
+        self.inv_freq = self.position.table if self.rot > 0 else None
+        self.layout, self.mscale = self.position.layout_code, self.position.mscale
+        self.gate_per_element = self._gate(spec) == "element"
         self.scale = spec.softmax_scale if spec.softmax_scale is not None else (self.dim + self.rot_dim) ** -0.5
         # the joint input projection: [dq | dkv (owners) | g], rows padded to a multiple of 16
         names = ["dq"] + (["dkv"] if self.owner else []) + ["g"]
@@ -127,16 +139,17 @@ class LatentAttention:
         T, H, dt = x.shape[0], self.H, self.ctx.dtype
         a = self.inp(x, out_dtype=self.inp.wide_dtype(T))
         cq, gate = K.latent_prep(a, self.q_off, self.q_rank, self.w_dq_norm, self.kv_off, self.kv_rank, self.rot_dim,
-                                 self.w_dkv_norm, self.g_off, H, self.eps, self.inv_freq, self.rot, batch.tok_pos,
+                                 self.w_dkv_norm, self.g_off, 0 if self.gate_per_element else H, self.eps, self.inv_freq, self.rot, batch.tok_pos,
                                  batch.tok_seq, kv.block_table, kv.page_size, kv.k if self.owner else None, self.row,
-                                 self.rank_pad, dt)
+                                 self.rank_pad, dt, layout=self.layout, mscale=self.mscale)
+        gates = a[:, self.g_off:self.g_off + H * self.vdim] if self.gate_per_element else None
         q = self.uq(cq)                                                   # [T, H * (dim + rot_dim)]
         hq = self.dim + self.rot_dim
         many = dt == torch.bfloat16 and T > MANY_ROWS                     # the per-head products go to the library
         ql = torch.empty((T, H * self.row), dtype=dt, device=x.device)    # per head [q^n Wuk | 0 | rope(q^r) | 0]
         K.head_gemm(q, H * hq, hq, None if many else self.w_uk, ql, H * self.row, self.row, T, H, self.dim,
                     self.kv_rank, rot_dim=self.rot_dim, rot=self.rot, inv_freq=self.inv_freq, tok_pos=batch.tok_pos,
-                    tail_off=self.rank_pad)
+                    tail_off=self.rank_pad, layout=self.layout, mscale=self.mscale)
         if many:
             # a product per head, written where the head's row of ql has its place (a strided view: no copy afterwards)
             torch.bmm(q.view(T, H, hq)[:, :, :self.dim].transpose(0, 1), self.w_uk,
@@ -147,16 +160,18 @@ class LatentAttention:
         if many:
             torch.bmm(ol.view(T, H, self.rank_pad)[:, :, :self.kv_rank].transpose(0, 1), self.w_uv,
                       out=o.view(T, H, self.vdim).transpose(0, 1))
-            if not gated:
+            if gates is not None:
+                K.sigmoid_mul(o, gates)
+            elif not gated:
                 o = (o.view(T, H, self.vdim) * gate[:, :, None]).to(dt).view(T, H * self.vdim)
         else:
             K.head_gemm(ol, H * self.rank_pad, self.rank_pad, self.w_uv, o, H * self.vdim, self.vdim, T, H,
-                        self.kv_rank, self.vdim, mul=None if gated else gate)
+                        self.kv_rank, self.vdim, mul=None if gated else gate, gate=gates)
         return self.o(o, out_dtype=self.o.wide_dtype(T))
 
-    def attend(self, ql: torch.Tensor, ol: torch.Tensor, batch, kv, gate: torch.Tensor) -> bool:
+    def attend(self, ql: torch.Tensor, ol: torch.Tensor, batch, kv, gate: Optional[torch.Tensor]) -> bool:
         """Attention of the step's tokens over the cached rows: ``H`` query heads on one row per key.  Returns
-        whether the gate is already in ``ol`` (a factor per (token, head) commutes with the head's value projection,
+        whether the gate per head (None: there is none) is already in ``ol`` (a factor per (token, head) commutes with the head's value projection,
         and the tensor-core kernel applies it as it writes)."""
         T = ql.shape[0]
         if K.attn_latent_supported(ql.dtype, self.row, self.rank_pad, kv.page_size):
@@ -177,7 +192,7 @@ class LatentAttention:
             scratch = batch.workspace.floats(K.attn_tokens_scratch_bytes(T, self.H, self.rank_pad, n) // 4)
         K.attn_tokens_kv(ql, ql.stride(0), ol, kv.k, kv.k, kv.block_table, batch.tok_pos, batch.tok_seq, T, self.H, 1,
                          self.row, self.rank_pad, self.row, kv.page_size, 0, self.scale, split, n, scratch)
-        return False
+        return gate is None
 
     def _chunks(self, batch, page: int, device):
         """``(pages per chunk, chunks)`` for the tensor-core kernel: one chunk when the step's tiles of rows already

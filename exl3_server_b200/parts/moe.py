@@ -20,8 +20,15 @@ score is the sum of its two largest choice scores), ``shared_inner`` (0: none); 
 ``expert`` = ``"clamped_glu"`` makes the experts (and the shared one) gated with a bounded gate, ``Wd (g sigmoid(alpha
 g) (u + 1))``, ``g = min(Wg r, limit)``, ``u = clamp(Wu r, -limit, limit)`` (tensors ``e<i>.gate``, ``e<i>.up``,
 ``e<i>.down``; parameters ``limit``, ``shared_limit``, ``alpha``): gate and up are one stacked matrix per expert, the
-activation a kernel of its own between the two grouped products.  Tensors: ``router [experts + identity, width]``, ``correction [experts + identity]`` and the
+activation a kernel of its own between the two grouped products.  ``expert`` = ``"glu"``: gated experts ``Wd (act(Wg r) *
+(Wu r))`` (the same tensor names); gate and up rows alternate in one stacked matrix, so that the activation is the first
+product's epilogue in all three of its kernels.  Tensors: ``router [experts + identity, width]``, ``correction [experts + identity]`` and the
 experts'.
+
+``table_routed``: there is no router.  An integer table ``table [vocab, top]`` gives every token id its ``top`` experts, each
+with the weight ``1 / top`` (parameters ``vocab``, ``experts``, ``top``, ``expert``, ``activation``).  The plans of all such
+layers of a model depend on the token ids alone: the first one that runs in a step has one kernel make them all
+(``kernels.moe_table_plans``), for every pass over a layer that runs several times too.
 
 How it runs (``csrc/moe.cu``): the router kernel also computes the shared expert's gate (its vector is one more row
 of the router's float32 matrix); a one-block kernel orders the step's (token, pick) pairs by expert into tiles, on the
@@ -71,6 +78,20 @@ class RoutedFeedForward:
     def _clamped(spec: FeedForwardSpec) -> bool:
         return spec.params.get("expert", "dense") == "clamped_glu"
 
+    @staticmethod
+    def _glu(spec: FeedForwardSpec) -> bool:
+        return spec.params.get("expert", "dense") == "glu"
+
+    @classmethod
+    def _expert_specs(cls, spec: FeedForwardSpec, prefix: str, n: int) -> List[TensorSpec]:
+        out = []
+        for e in range(n):
+            if cls._clamped(spec) or cls._glu(spec):
+                out.append(TensorSpec(f"{prefix}e{e}.gate", (spec.inner, spec.width)))
+            out += [TensorSpec(f"{prefix}e{e}.up", (spec.inner, spec.width)),
+                    TensorSpec(f"{prefix}e{e}.down", (spec.width, spec.inner))]
+        return out
+
     @classmethod
     def _shared_spec(cls, spec: FeedForwardSpec, inner: int) -> FeedForwardSpec:
         if cls._clamped(spec):
@@ -92,11 +113,7 @@ class RoutedFeedForward:
             out.append(TensorSpec(prefix + "correction", (E + I,)))
         if spec.params.get("router_bias", False):
             out.append(TensorSpec(prefix + "router.b", (E + I,)))
-        for e in range(E):
-            if cls._clamped(spec):
-                out.append(TensorSpec(f"{prefix}e{e}.gate", (spec.inner, spec.width)))
-            out += [TensorSpec(f"{prefix}e{e}.up", (spec.inner, spec.width)),
-                    TensorSpec(f"{prefix}e{e}.down", (spec.width, spec.inner))]
+        out += cls._expert_specs(spec, prefix, E)
         if shared:
             out += cls._shared_class(spec).tensor_specs(cls._shared_spec(spec, shared), prefix + "shared.")
             if spec.params.get("shared_gate", True):
@@ -112,10 +129,9 @@ class RoutedFeedForward:
         self.groups, self.keep = int(p.get("groups", 1)), int(p.get("keep", 1))
         self.act, self.score = p.get("activation", "gelu"), p.get("score", "softmax")
         self.group_score = p.get("group_score", "max")
-        self.clamped = self._clamped(spec)
-        if self.clamped:
-            self.act = "none"                  # the bounded gate is applied between the two products
-            self.limit, self.alpha = float(p["limit"]), float(p.get("alpha", ClampedGLU.ALPHA))
+        self._expert_form(spec)
+        if self.glu and shared:
+            raise ValueError("routed feed-forward: no shared expert beside experts of the form 'glu'")
         if self.act not in K.MOE_ACTIVATIONS or self.score not in K.MOE_SCORES or self.group_score not in K.MOE_GROUP_SCORES:
             raise ValueError(f"routed feed-forward: unknown activation {self.act!r}, score {self.score!r} or group "
                              f"score {self.group_score!r}")
@@ -141,20 +157,32 @@ class RoutedFeedForward:
             self.correction = torch.zeros(n, dtype=torch.float32, device=self.router.device)
         self.w_up = self.w_down = None
         if E:
-            if self.clamped:                   # [gate; up] rows of every expert
-                self.w_up = torch.stack([torch.cat([tensors[f"{prefix}e{e}.gate"].to(ctx.dtype),
-                                                    tensors[f"{prefix}e{e}.up"].to(ctx.dtype)], dim=0)
-                                         for e in range(E)]).contiguous()
-            else:
-                self.w_up = torch.stack([tensors[f"{prefix}e{e}.up"].to(ctx.dtype) for e in range(E)]).contiguous()
-            self.w_down = torch.stack([tensors[f"{prefix}e{e}.down"].to(ctx.dtype) for e in range(E)]).contiguous()
+            self._stack_experts(tensors, prefix, E, ctx)
+
+    def _expert_form(self, spec: FeedForwardSpec) -> None:
+        p = spec.params
+        self.clamped, self.glu = self._clamped(spec), self._glu(spec)
+        if self.clamped:
+            self.act = "none"                  # the bounded gate is applied between the two products
+            self.limit, self.alpha = float(p["limit"]), float(p.get("alpha", ClampedGLU.ALPHA))
+
+    def _stack_experts(self, tensors: Dict[str, torch.Tensor], prefix: str, E: int, ctx: BuildContext) -> None:
+        get = lambda e, name: tensors[f"{prefix}e{e}.{name}"].to(ctx.dtype)
+        if self.clamped:                       # [gate; up] rows of every expert
+            ups = [torch.cat([get(e, "gate"), get(e, "up")], dim=0) for e in range(E)]
+        elif self.glu:                         # gate and up rows in turn
+            ups = [torch.stack([get(e, "gate"), get(e, "up")], dim=1).reshape(-1, self.spec.width) for e in range(E)]
+        else:
+            ups = [get(e, "up") for e in range(E)]
+        self.w_up = torch.stack(ups).contiguous()
+        self.w_down = torch.stack([get(e, "down") for e in range(E)]).contiguous()
 
     def _pieces(self, x: torch.Tensor, batch):
         idx, wt, gate = K.moe_route(x, self.router, self.correction, self.E + self.I, self.gates,
                                     self.groups, self.keep, self.top, self.scale, self.score, self.group_score)
         y = None
         if self.E:
-            y = self._experts(x, idx)
+            y = self._experts(x, idx.numel(), lambda kind: K.moe_plan(idx, self.E, K.moe_tile_rows(kind)))
         s = self.shared.forward(x, batch) if self.shared is not None else None
         return y, idx, wt, s, gate
 
@@ -169,25 +197,31 @@ class RoutedFeedForward:
             return self.forward(x, batch)
         return PickedSum(*self._pieces(x, batch), n_experts=self.E)
 
-    def _experts(self, x: torch.Tensor, idx: torch.Tensor) -> torch.Tensor:
-        """float32 ``[pairs, width]``: every planned pair's expert output at the pair's own place."""
-        pairs = idx.numel()
+    def _product(self, pairs: int) -> str:
+        """Which of the experts' products (``kernels.moe_tile_rows``) takes a step of so many pairs."""
         width, inner = self.w_up.shape[2], self.w_down.shape[2]
-        glu = (lambda mid: K.clamped_glu(mid, self.limit, self.alpha, self.dtype)) if self.clamped else (lambda mid: mid)
-        vec = self.dtype == torch.bfloat16 and x.dtype == torch.bfloat16 and width % 8 == 0 and inner % 8 == 0 and \
-            x.stride(0) % 8 == 0
-        if vec and pairs >= MANY_PAIRS and K.moe_tc_supported(self.dtype, inner, width):
-            order, plan = K.moe_plan(idx, self.E, K.moe_tile_rows("tc"))
+        if self.dtype == torch.bfloat16 and width % 8 == 0 and inner % 8 == 0:
+            if pairs >= MANY_PAIRS and K.moe_tc_supported(self.dtype, inner, width):
+                return "tc"
+            if pairs <= FEW_PAIRS:
+                return "few"
+        return "tile"
+
+    def _experts(self, x: torch.Tensor, pairs: int, plan_for) -> torch.Tensor:
+        """float32 ``[pairs, width]``: every planned pair's expert output at the pair's own place.  ``plan_for(kind)``: the
+        step's ``(order, plan)`` with the tiles of that product."""
+        gated = (lambda mid: K.clamped_glu(mid, self.limit, self.alpha, self.dtype)) if self.clamped else (lambda mid: mid)
+        kind = self._product(pairs)
+        if kind != "tile" and (x.dtype != torch.bfloat16 or x.stride(0) % 8 != 0):
+            x = x.to(torch.bfloat16).contiguous()
+        order, plan = plan_for(kind)
+        if kind == "tc":
             xs = K.moe_gather(x, self.top, order, plan)
-            mid = glu(K.moe_gemm_tc(xs, self.w_up, order, plan, self.dtype, act=self.act))
+            mid = gated(K.moe_gemm_tc(xs, self.w_up, order, plan, self.dtype, act=self.act, glu=self.glu))
             return K.moe_gemm_tc(mid, self.w_down, order, plan, torch.float32)
-        if vec and pairs <= FEW_PAIRS:
-            order, plan = K.moe_plan(idx, self.E, K.moe_tile_rows("few"))
-            mid = glu(K.moe_gemv(x, self.top, self.w_up, order, plan, self.dtype, act=self.act))
-            return K.moe_gemv(mid, 1, self.w_down, order, plan, torch.float32)
-        order, plan = K.moe_plan(idx, self.E)
-        mid = glu(K.moe_gemm(x, self.top, self.w_up, order, plan, self.dtype, act=self.act))
-        return K.moe_gemm(mid, 1, self.w_down, order, plan, torch.float32)
+        product = K.moe_gemv if kind == "few" else K.moe_gemm
+        mid = gated(product(x, self.top, self.w_up, order, plan, self.dtype, act=self.act, glu=self.glu))
+        return product(mid, 1, self.w_down, order, plan, torch.float32)
 
     def untouched_bytes(self, tokens: int) -> int:
         """Bytes of experts' matrices that a step of ``tokens`` tokens is not expected to read when every router output
@@ -209,4 +243,52 @@ class RoutedFeedForward:
         return n
 
 
+class TableRoutedFeedForward(RoutedFeedForward):
+    @classmethod
+    def tensor_specs(cls, spec: FeedForwardSpec, prefix: str) -> List[TensorSpec]:
+        E, top = int(spec.params["experts"]), int(spec.params["top"])
+        return cls._expert_specs(spec, prefix, E) + \
+            [TensorSpec(prefix + "table", (int(spec.params["vocab"]), top), kind="int", high=E)]
+
+    def __init__(self, spec: FeedForwardSpec, tensors: Dict[str, torch.Tensor], prefix: str, ctx: BuildContext):
+        p = spec.params
+        self.spec, self.dtype = spec, ctx.dtype
+        self.E, self.I, self.top = int(p["experts"]), 0, int(p["top"])
+        self.act = p.get("activation", "silu")
+        self._expert_form(spec)
+        if self.act not in K.MOE_ACTIVATIONS or not 1 <= self.top <= self.E:
+            raise ValueError(f"table-routed feed-forward: activation {self.act!r}, {self.E} experts, top {self.top}")
+        self.shared = None
+        self.table = tensors[prefix + "table"].to(torch.int32).contiguous()
+        if self.table.numel() and not (0 <= int(self.table.min()) and int(self.table.max()) < self.E):
+            raise ValueError(f"{prefix}table: entries must lie below the {self.E} experts")
+        self._stack_experts(tensors, prefix, self.E, ctx)
+        # all layers of this kind in the model: their plans are made together
+        self.peers = ctx.shared.setdefault("table_routed", [])
+        self.place = len(self.peers)
+        self.peers.append((self.table, self.E, self.top, self._product))
+
+    def _plan(self, batch):
+        plans = batch.memo.get("table_routed")
+        if plans is None:
+            T = batch.token_ids.numel()
+            plans = batch.memo["table_routed"] = K.moe_table_plans(
+                batch.token_ids, [(table, E, K.moe_tile_rows(product(T * top))) for table, E, top, product in self.peers])
+        return plans[self.place]
+
+    def forward_picks(self, x: torch.Tensor, batch):
+        """``(y float32 [T * top, width], top, weight)``: the output is ``weight * sum_k y[t * top + k]``, which the caller's
+        next kernel adds up."""
+        return self._experts(x, x.shape[0] * self.top, lambda kind: self._plan(batch)), self.top, 1.0 / self.top
+
+    def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
+        out = torch.zeros((x.shape[0], self.spec.width), dtype=torch.float32, device=x.device)
+        K.residual_step(out, picks=self.forward_picks(x, batch))
+        return out
+
+    def weight_bytes(self) -> int:
+        return (self.w_up.numel() + self.w_down.numel()) * self.w_up.element_size()
+
+
 register_feed_forward("routed", RoutedFeedForward)
+register_feed_forward("table_routed", TableRoutedFeedForward)

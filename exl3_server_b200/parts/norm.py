@@ -108,6 +108,10 @@ class RMSNorm:
             return self._w32
         return self.weight
 
+    def rms_args(self):
+        """``(weight, eps, dtype of the output)`` for a kernel that applies this norm together with something else."""
+        return self.weight, self.spec.eps, self.out_dtype
+
     def fuse_args(self):
         """``(weight, eps, width)`` for a projection kernel that prepares this norm (see ``NormAfter``)."""
         return self.weight, self.spec.eps, self.spec.width

@@ -20,6 +20,8 @@ Per token ``q, k, v = r Wq^T, r Wk^T, r Wv^T`` (one joint matrix; biases optiona
 * ``softcap`` > 0: the scaled scores become ``softcap * tanh(score / softcap)``;
 * ``distance_bias``: the largest distance of a learned table ``rel [rows, heads]`` of score biases by distance (see
   ``parts/distance_bias.py``), added to the scores after scale and cap;
+* ``gate`` ``"head"``: head h's output is multiplied by ``sigmoid(Wg r)_h``, one number per head (tensor ``g``), before the
+  output projection;
 * ``reads_kv``: the layer has no keys and values of its own; its schedule entry names the entry whose cache it reads;
 * ``tile_rows``: in bfloat16, key and value rows of up to 64 (128) features are kept 64 (128) wide in the cache, the rest
   zeros, so that every such head size is the tensor-core kernels';
@@ -31,14 +33,14 @@ Per token ``q, k, v = r Wq^T, r Wk^T, r Wv^T`` (one joint matrix; biases optiona
 ``y = concat_h(o_h) Wo^T`` (+ bias).  Norms, rotation, mixing, scores and softmax are float32.  One kernel
 (``kernels.qk_prep``) does everything between the projection and the attention and writes the cache.  In bfloat16
 with keys and values of 64 or 128 features the attention is the tensor-core kernels' (tcgen05 for prompts, which
-takes every option above; the TMA page stream for steps of few tokens, which takes sinks, distance biases and the blocks
-but no window and no cap); everything else (float32,
+takes every option above; the TMA page stream for steps of few tokens, which takes all but caps and windows that keep the
+first keys); everything else (float32,
 other sizes, values of another width than keys) is the CUDA-core kernel in its general form
 (``kernels.attn_tokens_ex``), the same for prompts, portions of prompts and single tokens.  Head sizes are padded to
 a multiple of 8 in the cache (zeros), so any even size runs.
 
 Tensor names under the mixer's prefix: ``q``, ``k``, ``v``, ``o`` (biases: the name + ``.b``), ``q.norm``,
-``k.norm``, ``vmix``, ``sink``, ``rel``.
+``k.norm``, ``vmix``, ``sink``, ``rel``, ``g``.
 
 A mixer of this kind can also run on a slice of a projection that another part computed together with other
 inputs' (``input_weight`` / ``forward_projected``; see ``parts/parallel.py``).
@@ -91,6 +93,8 @@ class NormedAttention:
             out += [TensorSpec(prefix + n + ".b", (rows[n],)) for n in names]
             if spec.params["bias"] != "qkv":
                 out.append(TensorSpec(prefix + "o.b", (spec.width,)))
+        if spec.params.get("gate", "none") == "head":
+            out.append(TensorSpec(prefix + "g", (H, spec.width)))
         if spec.params.get("sink") == "learned":
             out.append(TensorSpec(prefix + "sink", (H,)))
         kind = spec.params.get("qk_norm", "none")
@@ -141,6 +145,17 @@ class NormedAttention:
         names = self._projected(spec)
         self._w = torch.cat([tensors[prefix + n].to(ctx.dtype) for n in names], dim=0)
         self._b = torch.cat([tensors[prefix + n + ".b"].to(ctx.dtype) for n in names]) if bias else None
+        self.gate_at: Optional[int] = None                  # column of the gates' logits behind the projection's first
+        if p.get("gate", "none") not in ("none", "head"):
+            raise ValueError(f"normed attention: gate must be 'none' or 'head', got {p.get('gate')!r}")
+        if p.get("gate", "none") == "head":
+            # the gates are rows of the joint matrix (zero rows up to a multiple of 16)
+            self.gate_at = self._w.shape[0]
+            pad = -(self.gate_at + H) % 16
+            zeros = lambda *shape: torch.zeros(shape, dtype=ctx.dtype, device=self._w.device)
+            self._w = torch.cat([self._w, tensors[prefix + "g"].to(ctx.dtype), zeros(pad, spec.width)], dim=0)
+            if self._b is not None:
+                self._b = torch.cat([self._b, zeros(H + pad)])
         self.n_proj = self._w.shape[0]
         self.qkv: Optional[Linear] = None                   # made on first use: a parallel part may project for us
         wo = tensors[prefix + "o"].to(ctx.dtype)
@@ -157,9 +172,9 @@ class NormedAttention:
         # positions bounds a query's keys as a window of that many keys does.
         self._cuts = Attention.__new__(Attention)
         self._cuts.spec = MixerSpec(kind="attention", width=spec.width, heads=H, kv_heads=G, head_dim=self.d_pad,
-                                    window=self.chunk or (self.window + self.keep_first if self.window else 0))
-        # what the decode kernel does not apply
-        self._plain_scores = self.window == 0 and self.softcap == 0.0
+                                   window=self.chunk or (self.window + self.keep_first if self.window else 0))
+        # what the decode kernel does not apply: caps, and windows beside kept first keys
+        self._plain_scores = self.keep_first == 0 and self.softcap == 0.0
 
     # -- what a part that projects for several mixers at once needs -----------------------------------------------
     def input_weight(self) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
@@ -194,13 +209,15 @@ class NormedAttention:
                 raise RuntimeError("normed attention: no earlier layer left its values to mix in")
             mix = (self.lam, src)
         own = not self.reads_kv
-        q, _ = K.qk_prep(proj, q_off, k_off if own else 0, v_off if own else -1, H, G if own else 0, d, dv, self.d_pad,
-                         self.dv_pad, self.norm, self.q_w, self.k_w, self.eps, self.rot, self.position.layout_code,
-                         self.position.table if self.rot else None, self.position.mscale, 1.0, mix, batch.tok_pos,
-                         batch.tok_seq, kv.block_table, kv.page_size, self.ctx.dtype, kv.k if own else None,
-                         kv.v if own else None, temperature=self.q_temp)
+        q, _, *gates = K.qk_prep(proj, q_off, k_off if own else 0, v_off if own else -1, H, G if own else 0, d, dv, self.d_pad,
+                                 self.dv_pad, self.norm, self.q_w, self.k_w, self.eps, self.rot, self.position.layout_code,
+                                 self.position.table if self.rot else None, self.position.mscale, 1.0, mix, batch.tok_pos,
+                                 batch.tok_seq, kv.block_table, kv.page_size, self.ctx.dtype, kv.k if own else None,
+                                 kv.v if own else None, temperature=self.q_temp,
+                                 gate_off=off + self.gate_at if self.gate_at is not None else None)
+        gate = gates[0] if gates else None
         out = torch.empty((T, H * self.dv_pad), dtype=self.ctx.dtype, device=proj.device)
-        if self._tensor_cores(q, out, batch, kv):
+        if self._tensor_cores(q, out, batch, kv, gate):
             return self.o(out, out_dtype=self.o.wide_dtype(T))
         split = max(SPLIT_KEYS, kv.page_size)
         if split % kv.page_size:
@@ -217,13 +234,13 @@ class NormedAttention:
         K.attn_tokens_ex(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.tok_pos, batch.tok_seq, T, H, G,
                          self.d_pad, self.dv_pad, kv.page_size, self.window, self.chunk, self.sink, self.scale, split, n,
                          scratch, keep_first=self.keep_first, softcap=self.softcap, sink_vals=self.sink_vals,
-                         dist=self.dist)
+                         dist=self.dist, gate=gate)
         return self.o(out, out_dtype=self.o.wide_dtype(T))
 
-    def _tensor_cores(self, q: torch.Tensor, out: torch.Tensor, batch, kv) -> bool:
+    def _tensor_cores(self, q: torch.Tensor, out: torch.Tensor, batch, kv, gate=None) -> bool:
         """bfloat16 with keys and values of 64 or 128 features: prompts through the tcgen05 kernel, steps of few
-        tokens through the kernel that streams pages by TMA, both with the sink and the blocks of positions as
-        parameters.  False when the sizes are not theirs (the CUDA-core kernel then takes the step)."""
+        tokens through the kernel that streams pages by TMA, both with the sink, the window, the blocks of positions
+        and the gate as parameters.  False when the sizes are not theirs (the CUDA-core kernel then takes the step)."""
         if self.ctx.dtype != torch.bfloat16 or self.d_pad != self.dv_pad:
             return False
         H, G, d, T = self.H, self.G, self.d_pad, q.shape[0]
@@ -236,10 +253,10 @@ class NormedAttention:
             K.attn_prefill_tc(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.row_start, batch.row_pos0, tile_seq,
                               tile_q0, n_tiles, H, G, d, kv.page_size, self.window, self.scale, variant=variant,
                               chunk=self.chunk, sink=self.sink, keep_first=self.keep_first, softcap=self.softcap,
-                              sink_vals=self.sink_vals, dist=self.dist)
+                              sink_vals=self.sink_vals, dist=self.dist, gate=gate)
             return True
         if not self._plain_scores:
-            return False                 # single tokens with a window or a cap: the CUDA-core kernel
+            return False                 # single tokens with a cap or kept first keys: the CUDA-core kernel
         if not K.attn_decode_supported(torch.bfloat16, T, H, G, d, kv.page_size, kv.page_size, 1):
             return False
         split, head_split, in_block = self._cuts._decode_split(T, batch.max_kv_len, kv.page_size, q.device)
@@ -249,8 +266,8 @@ class NormedAttention:
         if n > 1 and not in_block:
             scratch = batch.workspace.floats(K.attn_tokens_scratch_bytes(T, H, d, n) // 4)
         K.attn_decode(q, q.stride(0), out, kv.k, kv.v, kv.block_table, batch.tok_pos, batch.tok_seq, T, H, G, d,
-                      kv.page_size, 0, self.scale, split, n, scratch, head_split=head_split, in_block=in_block,
-                      twins=twins, chunk=self.chunk, sink=self.sink, sink_vals=self.sink_vals, dist=self.dist)
+                      kv.page_size, self.window, self.scale, split, n, scratch, head_split=head_split, in_block=in_block,
+                      twins=twins, chunk=self.chunk, sink=self.sink, sink_vals=self.sink_vals, dist=self.dist, gate=gate)
         return True
 
     def _chunks(self, max_kv_len: int, split: int) -> int:

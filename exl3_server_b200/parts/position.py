@@ -18,7 +18,10 @@ Parameters of a ``rope`` spec (``PositionSpec.params``), for mixers that apply t
 * ``yarn``: ``{"factor", "original", "fast", "slow"}``, a frequency table stretched for contexts beyond
   ``original`` positions: with ``n(t) = dims ln(original / (2 pi t)) / (2 ln theta)``, ``lo = max(floor(n(fast)), 0)``,
   ``hi = min(ceil(n(slow)), dims - 1)`` and ``ramp_d = clamp((d - lo) / max(hi - lo, 0.001), 0, 1)``, the frequency is
-  ``f_d / factor * ramp_d + f_d (1 - ramp_d)``, and sines and cosines are multiplied by ``0.1 ln(factor) + 1``.
+  ``f_d / factor * ramp_d + f_d (1 - ramp_d)``, and sines and cosines are multiplied by ``0.1 ln(factor) + 1``;
+* ``bands``: ``{"factor", "low", "high", "original"}``, frequencies scaled by bands of wavelengths ``l_d = 2 pi / f_d`` (as
+  the Llama 3.1 models do): ``f_d`` stays where ``l_d < original / high``, becomes ``f_d / factor`` where ``l_d > original /
+  low`` and in between ``(1 - s) f_d / factor + s f_d`` with ``s = (original / l_d - low) / (high - low)``.
 
 The Llama-family kernels (``rotate_and_store``, ``fused_rotation``) know the half layout without that factor only.
 
@@ -49,13 +52,15 @@ class RotaryPosition:
             raise ValueError(f"rope: layout must be 'half' or 'interleaved', got {layout!r}")
         self.layout_code = 1 if layout == "interleaved" else 0
         yarn = spec.params.get("yarn")
+        if yarn and spec.params.get("bands"):
+            raise ValueError("rope: 'yarn' and 'bands' are two ways of scaling the same frequencies")
         self.mscale = 0.1 * math.log(float(yarn["factor"])) + 1.0 if yarn else 1.0
         self.plain = self.layout_code == 0 and self.mscale == 1.0       # what the Llama-family kernels apply
         self.inv_freq = K.rotary_table(self.frequencies(spec) * float(spec.scale)).to(ctx.device)
 
     @staticmethod
     def frequencies(spec: PositionSpec) -> torch.Tensor:
-        """float64 ``theta^(-2d/dims)`` for d < dims / 2, stretched when the spec has ``yarn`` parameters."""
+        """float64 ``theta^(-2d/dims)`` for d < dims / 2, scaled when the spec has ``yarn`` or ``bands`` parameters."""
         d = torch.arange(0, spec.dims // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(float(spec.theta), dtype=torch.float64), -2.0 * d / max(1, spec.dims))
         yarn = spec.params.get("yarn")
@@ -69,6 +74,12 @@ class RotaryPosition:
             hi = min(math.ceil(turns(float(yarn["slow"]))), spec.dims - 1)
             ramp = torch.clamp((d - lo) / max(hi - lo, 0.001), 0.0, 1.0)
             f = f / factor * ramp + f * (1.0 - ramp)
+        bands = spec.params.get("bands")
+        if bands and spec.dims:
+            factor, low, high, original = (float(bands[k]) for k in ("factor", "low", "high", "original"))
+            turns = original * f / (2.0 * math.pi)                    # original / wavelength
+            s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+            f = torch.where(turns > high, f, torch.where(turns < low, f / factor, (1.0 - s) * f / factor + s * f))
         return f
 
     @property

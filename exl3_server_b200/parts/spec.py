@@ -10,12 +10,14 @@ reference's per-layer ``LayerPlan`` (src/model.h:40-45).
 ``ModelPlan.schedule`` is the order in which layers run.  It is data: an entry
 names the layer whose weights run, and optionally the earlier entry whose cache
 it reads instead of owning one, so a layer may run twice and a layer may read
-another layer's keys and values.
+another layer's keys and values.  An entry may also say what is added to the
+residual ahead of it (the embedding's output, a learned vector), as models do
+that run a group of layers several times.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
 
 
 @dataclass(frozen=True)
@@ -79,6 +81,10 @@ class LayerSpec:
 class ScheduleEntry:
     layer: int                            # index into ModelPlan.layers
     cache_from: Optional[int] = None      # schedule index whose cache this entry reads
+    # what joins the residual right before this entry's layer (a pass over a group of layers that runs several times):
+    # the embedding's output, and a row of the plan's ``entry_vectors``
+    add_embedding: bool = False
+    add_vector: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -118,6 +124,8 @@ class ModelPlan:
     # patterns (``fnmatch``) of tensor names that a checkpoint of this architecture may carry and the model
     # does not read; any other tensor the parts did not ask for is an error
     ignorable: List[str] = field(default_factory=list)
+    # the tensor of the vectors that schedule entries add (``add_vector`` counts its rows): (name, rows), or None
+    entry_vectors: Optional[Tuple[str, int]] = None
 
     def validate(self) -> None:
         n = len(self.layers)
@@ -126,6 +134,8 @@ class ModelPlan:
         for i, e in enumerate(self.schedule):
             if not 0 <= e.layer < n:
                 raise ValueError(f"plan: schedule[{i}] names layer {e.layer}, model has {n}")
+            if e.add_vector is not None and (self.entry_vectors is None or not 0 <= e.add_vector < self.entry_vectors[1]):
+                raise ValueError(f"plan: schedule[{i}] adds vector {e.add_vector}, which the plan does not have")
             if e.cache_from is not None:
                 if not 0 <= e.cache_from < i:
                     raise ValueError(

@@ -35,6 +35,8 @@ class TensorSpec:
     # a dimension of -1 in ``shape`` is whatever the checkpoint has (a size that no configuration key gives, such
     # as the rank of a low-rank pair); random weights take ``free_dim`` there
     free_dim: int = 16
+    # integer tables: random weights fill each row with that many different numbers below ``high`` (0: zeros)
+    high: int = 0
 
 
 _FLOATS = (torch.float16, torch.bfloat16, torch.float32, torch.float64)

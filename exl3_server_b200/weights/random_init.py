@@ -5,7 +5,8 @@ registered architecture.  Each tensor has its own generator seeded from the
 seed and the tensor's name, so a tensor's values do not depend on which other
 tensors exist.  Matrices are N(0, std); norm weights are ``1 + N(0, norm_std)``
 or, with ``norm_std=None``, N(0, std) like everything else; optional tensors
-(biases) are written only when ``with_optional`` is set.  The reference has no
+(biases) are written only when ``with_optional`` is set.  Integer tables whose spec has a ``high`` get rows of different
+numbers below it.  The reference has no
 such mode; its tests seed ``mt19937`` by hand (tests/mla_incremental_test.cpp:21-41).
 """
 from __future__ import annotations
@@ -36,7 +37,12 @@ def random_tensors(manifest: Sequence[TensorSpec], seed: int, std: float = 0.02,
         g.manual_seed(_tensor_seed(seed, spec.name))
         shape = tuple(spec.free_dim if d == -1 else d for d in spec.shape)
         if spec.kind == "int":
-            yield spec.name, torch.zeros(shape, dtype=torch.int32, device=device)
+            if spec.high > 0:
+                # a row's entries differ: the places of its largest of `high` random numbers
+                draw = torch.rand((*shape[:-1], spec.high), generator=g, dtype=torch.float32, device=device)
+                yield spec.name, draw.topk(shape[-1], dim=-1).indices.to(torch.int32)
+            else:
+                yield spec.name, torch.zeros(shape, dtype=torch.int32, device=device)
             continue
         x = torch.randn(shape, generator=g, dtype=torch.float32, device=device)
         if spec.init == "ones":
