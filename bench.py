@@ -32,7 +32,8 @@ decoder (lightning recurrences, differential attention over a window, dense and
 routed feed-forwards) and the Potodra decoder (a residual of four streams, attention over a window that keeps the first
 keys, matrix memories with exponential gates, a gated delta rule beside causal attention, dense and routed
 feed-forwards) and the Tunavik decoder (causal attention with distance biases, a sink and shared keys and values, routed
-feed-forwards) beside the Llama-family decoder at equal width, depth, head count and feed-forward width,
+feed-forwards) and the Soporax decoder (latent attention, attention over a window and causal attention with gates, each beside
+its feed-forward on one norm, experts from a table, layers that run twice) beside the Llama-family decoder at equal width, depth, head count and feed-forward width,
 with random weights: one prompt of
 ``--prefill-tokens`` tokens and decode steps at ``--batch`` and ``--context``,
 for each of the size pairs in ``DESIGN_SIZES`` (or the one named by
@@ -209,6 +210,29 @@ def tunavik_config(z):
     moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 2}, "shared": {"ff": z["ff"] // 4}}
     layers = [TunavikLayer("attention", dict(att, kv_from=i - 1 if i % 4 == 3 else None), dict(moe)) for i in range(z["layers"])]
     return TunavikConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, logit_scale=1.5, logit_softcap=30.0, layers=layers)
+
+
+def soporax_config(z):
+    """Soporax at one of the size pairs: as many layer runs as the other sides have layers, a quarter of them a second pass
+    over the same layers.  Layers repeat latent attention (the Rigitar side's sizes, a gate per output feature) + dense,
+    attention over a window of 1,024 positions with a sink + routed, causal attention with a gate per head + routed (both
+    with the other sides' heads); 16 experts, 2 a token from a table, gated, a quarter of the dense feed-forward's width."""
+    from exl3_server_b200.config.soporax import SoporaxConfig, SoporaxLayer
+    hd, lat = z["head_dim"], z["latent"]
+    heads = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": hd, "vdim": hd, "scale": hd ** -0.5}
+    kinds = [
+        ("latent_attention", dict(heads=z["heads"], scale=(lat["dim"] + lat["rot_dim"]) ** -0.5,
+                                  rot={"base": 10000.0, "dims": lat["rot_dim"],
+                                       "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}, **lat),
+         {"kind": "dense", "ff": z["ff"], "limit": 7.0}),
+        ("attention", dict(heads, mask={"size": 1024}), None),
+        ("attention_2", dict(heads, rot={"base": 500000.0, "dims": hd,
+                                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}), None)]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 2}}
+    twice = z["layers"] // 4
+    layers = [SoporaxLayer(k, dict(m), dict(f or moe)) for k, m, f in (kinds[i % 3] for i in range(z["layers"] - twice))]
+    return SoporaxConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, logit_scale=0.5,
+                         loop={"start": 1, "stop": 1 + twice, "times": 2}, layers=layers)
 
 
 def design_configs(name: str):
@@ -436,7 +460,7 @@ class Rig:
 
 
 def designs(args) -> int:
-    """``--only designs``: prefill and decode throughput of the Rigitar, Nikodra, Nibelix, Potodra and Tunavik decoders beside
+    """``--only designs``: prefill and decode throughput of the Rigitar, Nikodra, Nibelix, Potodra, Tunavik and Soporax decoders beside
     the Llama-family decoder of equal sizes; one JSON line."""
     import torch
     torch.cuda.set_device(0)
@@ -450,7 +474,7 @@ def designs(args) -> int:
     for name in ([args.design_sizes] if args.design_sizes else sorted(DESIGN_SIZES)):
         rig_cfg, llama_cfg = design_configs(name)
         rec = {}
-        for arch, cfg in (("tunavik", tunavik_config(DESIGN_SIZES[name])), ("potodra", potodra_config(DESIGN_SIZES[name])), ("nibelix", nibelix_config(DESIGN_SIZES[name])),
+        for arch, cfg in (("soporax", soporax_config(DESIGN_SIZES[name])), ("tunavik", tunavik_config(DESIGN_SIZES[name])), ("potodra", potodra_config(DESIGN_SIZES[name])), ("nibelix", nibelix_config(DESIGN_SIZES[name])),
                           ("nikodra", nikodra_config(DESIGN_SIZES[name])),
                           ("rigitar", rig_cfg), ("llama", llama_cfg)):
             if args.design_arch not in ("both", arch):
@@ -493,7 +517,7 @@ def main() -> int:
                     help="run one part only (for profiling small cases); prints a short JSON line")
     ap.add_argument("--design-sizes", choices=sorted(DESIGN_SIZES), default=None,
                     help="with --only designs: one size pair instead of all")
-    ap.add_argument("--design-arch", choices=["both", "tunavik", "potodra", "nibelix", "nikodra", "rigitar", "llama"], default="both",
+    ap.add_argument("--design-arch", choices=["both", "soporax", "tunavik", "potodra", "nibelix", "nikodra", "rigitar", "llama"], default="both",
                     help="with --only designs: one of the designs only (both: all of them)")
     ap.add_argument("--design-part", choices=["both", "prefill", "decode"], default="both",
                     help="with --only designs: one of the two measurements only")

@@ -1,7 +1,7 @@
 """A plain, slow implementation of the Soporax decoder: whole sequences, no cache, float64, one function per mechanism.
 It shares no code with the package: config.json is read with ``json``, the weights with the ``safetensors`` library, and
 everything is plain torch arithmetic on the CPU.  Attention builds the full score matrix head by head with its mask; the
-latent attention forms every head's keys and values; experts are a loop over tokens.
+latent attention forms every head's keys and values; experts run one by one on the tokens whose rows list them.
 """
 from __future__ import annotations
 
@@ -71,12 +71,12 @@ def ramped_frequencies(dims: int, base: float, s: Optional[dict]):
 def rotate_neighbours(x: torch.Tensor, freqs: List[float], mult: float = 1.0) -> torch.Tensor:
     """x [T, ..., n]: features 2i and 2i + 1 of the first 2 len(freqs) turned by position times frequency i."""
     y = x.clone()
-    for p in range(x.shape[0]):
-        for i, f in enumerate(freqs):
-            c, s = mult * math.cos(p * f), mult * math.sin(p * f)
-            u, v = x[p, ..., 2 * i], x[p, ..., 2 * i + 1]
-            y[p, ..., 2 * i] = u * c - v * s
-            y[p, ..., 2 * i + 1] = v * c + u * s
+    at = torch.arange(x.shape[0], dtype=F).view(-1, *[1] * (x.dim() - 2))
+    for i, f in enumerate(freqs):
+        c, s = mult * torch.cos(at * f), mult * torch.sin(at * f)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        y[..., 2 * i] = u * c - v * s
+        y[..., 2 * i + 1] = v * c + u * s
     return y
 
 
@@ -161,17 +161,17 @@ def clamped_feed_forward(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, li
 
 
 def expert(x: torch.Tensor, w: Dict[str, torch.Tensor], p: str) -> torch.Tensor:
-    z = w[p + "gate"] @ x
-    return w[p + "down"] @ (z * torch.sigmoid(z) * (w[p + "up"] @ x))
+    z = x @ w[p + "gate"].T
+    return (z * torch.sigmoid(z) * (x @ w[p + "up"].T)) @ w[p + "down"].T
 
 
 def experts_by_table(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, tokens: List[int]) -> torch.Tensor:
     """The mean of the experts that the token's row of the table lists."""
     out = torch.zeros_like(h)
-    for t, tok in enumerate(tokens):
-        picks = w[p + "table"][tok].tolist()
-        for e in picks:
-            out[t] += expert(h[t], w, f"{p}e{e}.") / len(picks)
+    rows = [w[p + "table"][tok].tolist() for tok in tokens]
+    for e in sorted({e for picks in rows for e in picks}):
+        at = [t for t, picks in enumerate(rows) if e in picks]
+        out[at] += expert(h[at], w, f"{p}e{e}.") / len(rows[0])
     return out
 
 
