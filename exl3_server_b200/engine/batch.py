@@ -73,6 +73,9 @@ class StepBatch:
     tile_keys: Dict[int, List[int]] = field(default_factory=dict)
     host_slots: List[int] = field(default_factory=list)
     host_new: List[int] = field(default_factory=list)
+    # a second stream, in steps of one token per sequence: a block whose two sublayers do not depend on each other may run
+    # one of them there (and must have joined it before it returns)
+    side: Optional[Any] = None
     # what a part has worked out for this step and wants to find again in the next layer (keyed as it likes)
     memo: Dict[Any, Any] = field(default_factory=dict)
 

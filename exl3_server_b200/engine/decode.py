@@ -81,6 +81,7 @@ class DecodeRunner:
         self.tok_seq = torch.arange(rows, dtype=torch.int32, device=dev)
         self.row_start = torch.arange(rows + 1, dtype=torch.int32, device=dev)
         self.next_ids = torch.zeros(rows, dtype=torch.int32, device=dev)
+        self.side = torch.cuda.Stream(device=dev)
         self.workspace = Workspace(dev, keep_outgrown=True)   # graphs keep the addresses they were recorded with
         self.graphs: Dict[int, torch.cuda.CUDAGraph] = {}
         self.graph_logits: Dict[int, torch.Tensor] = {}
@@ -111,7 +112,7 @@ class DecodeRunner:
             tok_seq=self.tok_seq, slot_ids=self.pad_slots if padding else self.slot_ids.dev,
             row_start=self.row_start, row_pos0=pos, want_rows=self.tok_seq, n_wanted=self.rows,
             block_tables=self.pad_tables if padding else [t.dev for t in self.tables],
-            max_kv_len=max_kv_len, max_new=1, workspace=self.workspace)
+            max_kv_len=max_kv_len, max_new=1, workspace=self.workspace, side=self.side)
 
     def _record(self, bucket: int) -> None:
         model, cache = self.engine.model, self.engine.cache

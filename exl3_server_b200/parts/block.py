@@ -226,16 +226,29 @@ class ParallelBlock:
         """The norms this block applies to the residual it is given."""
         return (self.mixer_norm,)
 
+    def _feed(self, r: torch.Tensor, batch):
+        """``(output, picks)`` of the feed-forward, one of them None."""
+        if self.feed_forward is None:
+            return None, None
+        if hasattr(self.feed_forward, "forward_picks"):
+            return None, self.feed_forward.forward_picks(r, batch)     # the sum over the picks is the step's kernel's
+        return self.feed_forward.forward(r, batch), None
+
     def forward(self, stream: ResidualStream, batch, kv, state, next_block=None, entry=None) -> None:
         left = stream.take_for(self.input_norms())
         r = left[0] if left is not None else self.mixer_norm.add_norm(stream)
-        y = self.mixer.forward(r, batch, kv, state)
-        b = picks = None
-        if self.feed_forward is not None:
-            if hasattr(self.feed_forward, "forward_picks"):
-                picks = self.feed_forward.forward_picks(r, batch)     # the sum over the picks is the step's kernel's
-            else:
-                b = self.feed_forward.forward(r, batch)
+        side = getattr(batch, "side", None) if self.feed_forward is not None else None
+        if side is not None:
+            # single tokens: neither sublayer fills the GPU, so the feed-forward runs beside the mixer on a second stream
+            main = torch.cuda.current_stream()
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                b, picks = self._feed(r, batch)
+            y = self.mixer.forward(r, batch, kv, state)
+            main.wait_stream(side)
+        else:
+            y = self.mixer.forward(r, batch, kv, state)
+            b, picks = self._feed(r, batch)
         nxt = next_block.input_norms() if hasattr(next_block, "input_norms") else ()
         fused = len(nxt) == 1 and hasattr(nxt[0], "rms_args")
         x = K.residual_step(stream.h, y, b, picks, float(self.spec.residual_scale), entry,

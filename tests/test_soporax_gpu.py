@@ -396,6 +396,27 @@ def test_the_batch_and_the_pages_change_nothing_in_float32(folders, name):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_the_second_stream_changes_nothing(folders, name, dtype, monkeypatch):
+    """Decode steps with the feed-forward beside the mixer on a second stream and with both in turn on one: the same bits."""
+    from exl3_server_b200.engine.decode import DecodeRunner
+    reqs = requests_for(name, [80, 33, 5], seed=47)
+    steps = batched_trace(reqs, [["r0", "r1", "r2"]], {"r0": 40, "r1": 2, "r2": 1})
+    with_side = run_trace(engine_for(folders[name], dtype), steps)
+    make = DecodeRunner._batch
+
+    def without(self, *args, **kwargs):
+        batch = make(self, *args, **kwargs)
+        assert batch.side is not None
+        batch.side = None
+        return batch
+    monkeypatch.setattr(DecodeRunner, "_batch", without)
+    alone = run_trace(engine_for(folders[name], dtype), steps)
+    for rid in reqs:
+        assert np.array_equal(with_side[rid], alone[rid]), rid
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["mixed", "odd", "wide"])
 def test_long_decoding(folders, name, dtype):
     """Three tokens of prompt, then 200 decoded one by one over three page borders and past most windows, two
