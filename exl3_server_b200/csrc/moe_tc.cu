@@ -41,7 +41,7 @@ static __device__ int g_mt_error = 0;
 __device__ inline float mt_act(float v, int act) {
   if (act == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
   if (act == 2) return 0.5f * v * (1.0f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
-  if (act == 3) return v / (1.0f + expf(-v));
+  if (act == 3) return __fdividef(v, 1.0f + __expf(-v));   // 1e-6 of the value; results are rounded to 16 bits or weighted
   if (act == 4) { const float r = fmaxf(v, 0.0f); return r * r; }
   return v;
 }
